@@ -120,7 +120,7 @@ __device__ __forceinline__ void mbar_wait(uint64_t* bar, uint32_t parity) {
     while (!mbar_try_wait(bar, parity)) {
     }
 }
-// 1-D bulk copy (TMA engine, SASS UBLKCP): bytes % 16 == 0, src/dst 16-B aligned.
+// 1-D bulk copy (TMA engine): bytes % 16 == 0, src/dst 16-B aligned.
 __device__ __forceinline__ void bulk_g2s(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
     asm volatile(
         "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
