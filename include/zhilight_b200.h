@@ -416,7 +416,8 @@ enum {
     ZL_GEMM_EPI_GEGLU_TANH = 5 /* columns 2j, 2j+1 = gate, up -> column j: gelu_tanh(gate) * up, with
                                   gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) */,
     ZL_GEMM_EPI_GELU_TANH_MUL = 6 /* gelu_tanh(v) * mul[m][n] */,
-    ZL_GEMM_EPI_SOFTCAP = 7 /* limit * tanh(v / limit) */
+    ZL_GEMM_EPI_SOFTCAP = 7 /* limit * tanh(v / limit) */,
+    ZL_GEMM_EPI_REGLU = 8 /* columns 2j, 2j+1 = gate, up -> column j: max(gate, 0) * up */
 };
 /* y[b](M,N) = epi(x[b](M,K) @ w[b](N,K)^T), b < batch, element strides per batch entry; any M, N, K.  in_dtype
  * ZL_F16 / ZL_BF16 (tensor cores, fp32 accumulation) or ZL_F32 (plain fp32 FMAs, no reduced-precision mode);
@@ -666,6 +667,14 @@ int zl_moe_route_grouped(const float* x, long long ldx, const float* w_router, c
                          float* top_weights, int32_t* group_offsets, int32_t* list_token, int32_t* list_pair, int T, int D,
                          int slots, int top, int groups, int keep, int score_fn, int renormalize, float renorm_eps, int pdl,
                          zl_stream_t stream);
+/* zl_moe_route_grouped with the router's input and weights in `in_dtype` (the dot products accumulate in fp32; fp32 with
+ * w_router NULL), a choice of how a group ranks -- its largest score + correction, or the sum of its two largest -- and the
+ * weights, after the renormalisation, times weight_scale. */
+enum { ZL_MOE_GROUP_MAX = 0, ZL_MOE_GROUP_TOP2 = 1 };
+int zl_moe_route_ex(const void* x, long long ldx, const void* w_router, int in_dtype, const float* correction,
+                    int32_t* top_experts, float* top_weights, int32_t* group_offsets, int32_t* list_token, int32_t* list_pair,
+                    int T, int D, int slots, int top, int groups, int keep, int group_rank, int score_fn, int renormalize,
+                    float renorm_eps, float weight_scale, int pdl, zl_stream_t stream);
 /* cos / sin of pos[t] * inv_freq[i] (double angles, evaluated in double) -> table (T, half) of float pairs (cos, sin). */
 int zl_rope_table(const int32_t* pos, int T, const double* inv_freq, int half, float* table, int pdl, zl_stream_t stream);
 enum { ZL_ROT_HALVES = 0 /* pair (i, i + n / 2) */, ZL_ROT_ADJACENT = 1 /* pair (2i, 2i + 1) */ };
@@ -699,6 +708,59 @@ int zl_gated_parallel_combine(float* x, long long ldx, float mult, const float* 
                               const float* coef, const int32_t* choice, int n_parts, int n_real, const float* f_dense,
                               long long ldf, int gf_off, const float* scale_f, const float* norm_w, const float* next_w,
                               void* h_next, int act_dtype, int T, int D, float eps, int pdl, zl_stream_t stream);
+/* The residual update of a pre-norm layer: x[t] += sum_p coef[t][p] * parts[t * n_parts + p] (coef NULL: ones; parts NULL: x
+ * stays).  next_w != NULL: next_w * x[t] / sqrt(mean(x[t]^2) + eps) of the new x -> h (T, D) of act_dtype; x_copy != NULL: the
+ * new x itself in act_dtype, rows ld_copy apart (the input of a Linear that reads the stream). */
+int zl_residual_norm(float* x, long long ldx, const float* parts, long long ldp, const float* coef, int n_parts,
+                     const float* next_w, void* h, void* x_copy, long long ld_copy, int act_dtype, int T, int D, float eps,
+                     int pdl, zl_stream_t stream);
+/* x[t] = table[ids[t]] (table (vocab, D) of act_dtype, x fp32), with the same outputs and a second copy. */
+int zl_embed_norm(const int32_t* ids, const void* table, int vocab, float* x, const float* next_w, void* h, void* x_copy,
+                  void* x_copy2, long long ld_copy, int act_dtype, int T, int D, float eps, int pdl, zl_stream_t stream);
+/* Rotation frequencies f_i = base^(-2i/dims), i < dims/2, scaled by wavelength when factor > 0: with l = 2 pi / f, f stays
+ * where l < original / high, becomes f / factor where l > original / low, and (1 - s) f / factor + s f with
+ * s = (original / l - low) / (high - low) between the two.  Host function; out (dims/2) doubles. */
+int zl_rope_inv_freq_wavelength(double base, int dims, double factor, double low, double high, double original, double* out);
+/* Attention in a sliding window over per-slot caches, an ordinary softmax: token t sees the keys j with
+ * 0 <= pos[t] - j < window (window 0: all j <= pos[t]).  maps = 1: q (T, heads, dim), keys (max_seq, kv_heads, dim), values
+ * (max_seq, kv_heads, vdim), out[t][h] = sum_j p_j v_j.  maps = 2 (differential attention): q (T, heads, 2, dim), keys
+ * (max_seq, kv_heads, 2, dim): each map m has its own softmax over q_m . k_m, both over the same values, and
+ * o = a_1 - lambda a_2, out[t][h] = out_mul * o / sqrt(mean(o^2) + out_eps).  gate != NULL: fp32 logits,
+ * out[t][h * vdim + c] times sigmoid(gate[t * ldg + h * vdim + c]).  out (T, heads * vdim) of `dtype`.  Splits and runs as in
+ * zl_sink_attention (splits of zl_sink_attention_splits with max_len at most the window; workspace for heads * maps). */
+int zl_window_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot, const int32_t* pos,
+                        float scale, int window, int maps, float lambda, float out_eps, float out_mul, const float* gate,
+                        long long ldg, void* out, int T, int heads, int kv_heads, int dim, int vdim, int splits,
+                        void* workspace, size_t workspace_bytes, const int32_t* run_row0, const int32_t* run_len, int runs,
+                        int max_run_len, int dtype, int pdl, zl_stream_t stream);
+/* Attention whose heads' scores are mixed before the softmax: s'_h = sum_g mix[h * heads + g] (q_g . k_{g / (heads / kv_heads)})
+ * (mix fp32 (heads, heads), the scores' scale folded in), ordinary softmax of s'_h over the visible keys (window as above),
+ * out[t][h] = sum_j p_j v_{h / (heads / kv_heads)}.  Same caches, splits (zl_mixed_head_attention_splits) and runs;
+ * workspace of zl_sink_attention_workspace_bytes. */
+int zl_mixed_head_attention_splits(int T, int heads, int max_len);
+int zl_mixed_head_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot, const int32_t* pos,
+                            const float* mix, int window, void* out, int T, int heads, int kv_heads, int dim, int vdim,
+                            int splits, void* workspace, size_t workspace_bytes, const int32_t* run_row0,
+                            const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl, zl_stream_t stream);
+/* From a fused projection row proj[t] (fp32) to the operands of absorbed latent attention with a rotated part: query head h
+ * (columns q_off + h * (dim + rot_dim)): its first `dim` columns -> q_out (T, heads, dim) of `dtype`, its last rot_dim ones
+ * turned by table[t] (adjacent pairs) -> columns rank_cols .. + rot_dim of qa[t][h] (fp32, row stride row_cols); columns
+ * c_off .. + kv_rank: RMS norm times kv_weight -> columns 0 .. of row pos[t] of slot_addrs[slot[t]] (row stride row_cols, of
+ * `dtype`), the rot_dim columns after them, turned alike -> its columns rank_cols .. + rot_dim.  Columns kv_rank .. rank_cols
+ * and rank_cols + rot_dim .. row_cols are padding that is never written. */
+int zl_latent_rope_append(const float* proj, long long ldp, int q_off, int heads, int dim, int rot_dim, const float* table,
+                          void* q_out, float* qa, int c_off, int kv_rank, const float* kv_weight, int rank_cols, int row_cols,
+                          void* const* slot_addrs, const int32_t* slot, const int32_t* pos, int T, float eps, int dtype, int pdl,
+                          zl_stream_t stream);
+/* zl_latent_attention over rows of row_cols columns of which all enter the score and the first rank_cols are the value:
+ * q_absorbed (T, heads, row_cols) fp32, out (T, heads, rank_cols) of `dtype`.  sink NULL: an ordinary softmax.
+ * gate != NULL: head h's output times sigmoid(gate[t * ldg + h]).  The probabilities enter the 16-bit product as a hi + lo
+ * pair.  Workspace and splits as for kv_rank = rank_cols. */
+int zl_latent_attention_prepare_ex(int heads, int rank_cols, int row_cols, int dtype);
+int zl_latent_attention_ex(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                           const float* sink, const float* gate, long long ldg, float scale, void* out, int T, int heads,
+                           int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes, int dtype, int pdl,
+                           zl_stream_t stream);
 /* ------------------------------------------------------------------------------------------ *
  * Kodupel: decoder-only model whose layers are listed one by one: the mixer is attention (grouped key/value heads,
  * biased projections, per-head query / key RMS norm, partial rotation in adjacent pairs with YaRN frequencies, value
@@ -839,6 +901,59 @@ int zl_dizizen_stats(zl_dizizen_t* m, double* weight_bytes, int* kernels_per_ste
 /* Copies rows 0 .. n_rows of one slot's key and value caches of a layer that owns them to the host as fp32:
  * keys (n_rows, kv_heads * dim), values (n_rows, kv_heads * vdim) (tests). */
 int zl_dizizen_read_cache(zl_dizizen_t* m, int layer, int slot, int n_rows, float* keys_host, float* values_host);
+
+/* ------------------------------------------------------------------------------------------ *
+ * Dekalorn: decoder-only model of pre-norm layers (RMS norm with plain weight) on an fp32 residual stream, listed one by
+ * one, of which a range may be looped: it runs loop_times times with the same weights, each pass with caches of its own
+ * and after x <- W_in [x; x0], x0 the token's embedding.  The mixer is latent attention with a rotated key part shared by
+ * the heads and a sigmoid gate per head, differential attention in a sliding window with a full-width sigmoid gate, or
+ * rotated attention in a sliding window whose heads' scores are mixed before the softmax.  The feed-forward is absent, a
+ * dense relu-gated unit, or a mixture of silu-gated experts chosen by sigmoid scores inside the groups whose two best
+ * scores sum highest.  Same driver shape as zl_dizizen_*.
+ * ------------------------------------------------------------------------------------------ */
+enum { ZL_DEKALORN_LATENT = 0, ZL_DEKALORN_DIFF = 1, ZL_DEKALORN_MIXED = 2 };
+typedef struct zl_dekalorn zl_dekalorn_t;
+typedef struct zl_dekalorn_layer {
+    int type;              /* ZL_DEKALORN_* */
+    int heads, kv_heads, dim, vdim; /* differential attention: dim is the size of one map */
+    int rot_dim, kv_rank;  /* latent attention: rotated part of a head, latent size */
+    int window;            /* sliding window, 0: none */
+    int rot_dims;          /* rotated dimensions of a head (latent attention: rot_dim) */
+    float scale, diff;     /* score scale; constant of the differential layer */
+    double rot_base, rot_factor /* 0: frequencies are not scaled */, rot_low, rot_high, rot_original;
+    int ff_kind;           /* ZL_FF_* */
+    int ff;                /* inner size of the dense feed-forward or of one expert */
+    int experts, top, groups, keep;
+    float router_scale;
+} zl_dekalorn_layer_t;
+typedef struct zl_dekalorn_config {
+    int num_layers, width, vocab;
+    float eps;
+    int loop_start, loop_stop, loop_times; /* loop_times 0: no loop */
+    int dtype; /* ZL_BF16 or ZL_F32 */
+    int max_batch, max_seq, max_step_tokens;
+    int use_pdl, use_graph;
+} zl_dekalorn_config_t;
+int zl_dekalorn_create(const zl_dekalorn_config_t* cfg, const zl_dekalorn_layer_t* layers, zl_dekalorn_t** out);
+void zl_dekalorn_destroy(zl_dekalorn_t* m);
+int zl_dekalorn_load_tensor(zl_dekalorn_t* m, const char* name, const void* data_host, int rows, int cols, int elem_bytes);
+int zl_dekalorn_init_synthetic(zl_dekalorn_t* m, uint64_t seed);
+int zl_dekalorn_finalize(zl_dekalorn_t* m);
+/* As zl_dekipel_step. */
+int zl_dekalorn_step(zl_dekalorn_t* m, const int32_t* tokens_host, const int32_t* slots_host, const int32_t* positions_host,
+                     int T, const int32_t* want_rows_host, int n_want, float* logits_host, int32_t* next_host);
+int zl_dekalorn_set_state(zl_dekalorn_t* m, const int32_t* tokens_host, const int32_t* positions_host, int B);
+int zl_dekalorn_step_device(zl_dekalorn_t* m, int B);
+int zl_dekalorn_sync(zl_dekalorn_t* m);
+zl_stream_t zl_dekalorn_stream(zl_dekalorn_t* m);
+/* residual stream after every layer run of the last step, (runs, T, width) fp32, when capture was switched on */
+int zl_dekalorn_capture_layers(zl_dekalorn_t* m, int on);
+int zl_dekalorn_read_layers(zl_dekalorn_t* m, float* out_host, int T);
+int zl_dekalorn_stats(zl_dekalorn_t* m, double* weight_bytes, int* kernels_per_step);
+/* Rows 0 .. n_rows of what layer run `run` caches for one slot, as fp32 (tests): latent attention: latents (n_rows, kv_rank)
+ * and rotated key parts (n_rows, rot_dim); otherwise keys (n_rows, kv_heads * dim, twice that for differential attention)
+ * and values (n_rows, kv_heads * vdim). */
+int zl_dekalorn_read_cache(zl_dekalorn_t* m, int run, int slot, int n_rows, float* a_host, float* b_host);
 #ifdef __cplusplus
 }
 #endif

@@ -1,7 +1,7 @@
 // General tiled GEMM y[b](M,N) = epi(x[b](M,K) @ w[b](N,K)^T) for any M, N, K, with a batch of strided problems
 // (one per attention head) and small fused epilogues: a per-column bias, relu^2, tanh, a sigmoid gate, the tanh form of
 // gelu times a per-element multiplier, a tanh soft cap, and gated units over column pairs (columns 2j / 2j+1 hold
-// gate / up, output column j): the clamped unit of expert feed-forwards and gelu_tanh(gate) * up.  Grouped mode serves
+// gate / up, output column j): the clamped unit of expert feed-forwards, gelu_tanh(gate) * up and relu(gate) * up.  Grouped mode serves
 // mixtures of experts: problem b owns the rows grp_off[b] .. grp_off[b+1] of a list sorted by expert, input rows are
 // gathered and output rows scattered through index lists, so one launch covers every expert of a step whatever
 // the routing turned out to be (the counts stay on the device: the launch can sit in a CUDA graph).
@@ -32,12 +32,12 @@ struct GemmP {
     int act_tanh = 0;                 // few-rows kernel without the gated unit: tanh of the (biased) sum
     float limit = 0.f, alpha = 1.f, beta = 0.f;   // gated unit: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(alpha g) (u + beta)
                                       // soft cap: limit * tanh(v / limit)
-    int pair_gelu = 0;                // few-rows kernel with a gated unit: gelu_tanh(gate) * up instead of the clamped unit
+    int pair_fn = ZL_GEMM_EPI_GLU_CLAMP;   // few-rows kernel with a gated unit: which of the pair epilogues
     int act_gelu_mul = 0;             // few-rows kernel without the gated unit: gelu_tanh of the (biased) sum times gate[m][n]
     int act_relu2 = 0;                // few-rows kernel without the gated unit: max(sum, 0)^2
 };
 
-__host__ __device__ constexpr bool epi_pairs(int epi) { return epi == ZL_GEMM_EPI_GLU_CLAMP || epi == ZL_GEMM_EPI_GEGLU_TANH; }
+__host__ __device__ constexpr bool epi_pairs(int epi) { return epi == ZL_GEMM_EPI_GLU_CLAMP || epi == ZL_GEMM_EPI_GEGLU_TANH || epi == ZL_GEMM_EPI_REGLU; }
 
 
 // rows of problem b and the place of its first row in the sorted list
@@ -58,6 +58,7 @@ __device__ __forceinline__ float glu_clamp(float gate, float up, const GemmP& p)
 template <int EPI>
 __device__ __forceinline__ float pair_unit(float gate, float up, const GemmP& p) {
     if constexpr (EPI == ZL_GEMM_EPI_GEGLU_TANH) return gelu_f(gate) * up;
+    else if constexpr (EPI == ZL_GEMM_EPI_REGLU) return fmaxf(gate, 0.f) * up;
     else return glu_clamp(gate, up, p);
 }
 
@@ -380,7 +381,7 @@ __global__ void __launch_bounds__(256) k_gemm_grouped_small(GemmP p) {
             float v = warp_sum(acc[m]), v2 = warp_sum(acc2[m]);
             if (GLU) {
                 if (p.bias) v += p.bias[(size_t)b * p.bb + 2 * n], v2 += p.bias[(size_t)b * p.bb + 2 * n + 1];
-                v = p.pair_gelu ? gelu_f(v) * v2 : glu_clamp(v, v2, p);
+                v = p.pair_fn == ZL_GEMM_EPI_GEGLU_TANH ? gelu_f(v) * v2 : (p.pair_fn == ZL_GEMM_EPI_REGLU ? fmaxf(v, 0.f) * v2 : glu_clamp(v, v2, p));
             } else {
                 if (p.bias) v += p.bias[(size_t)b * p.bb + n], v2 += has2 ? p.bias[(size_t)b * p.bb + n2] : 0.f;
                 if (p.act_tanh) v = tanhf(v), v2 = tanhf(v2);
@@ -518,6 +519,7 @@ static cudaError_t launch_mma(const GemmP& p, int batch, int epi, bool vx, bool 
         return launch(k_gemm_mma<T, TO, ZL_GEMM_EPI_GLU_CLAMP>, grid, block, 0, st, pdl, p, (int)vx, (int)vw);
     if (epi == ZL_GEMM_EPI_GEGLU_TANH)
         return launch(k_gemm_mma<T, TO, ZL_GEMM_EPI_GEGLU_TANH>, grid, block, 0, st, pdl, p, (int)vx, (int)vw);
+    if (epi == ZL_GEMM_EPI_REGLU) return launch(k_gemm_mma<T, TO, ZL_GEMM_EPI_REGLU>, grid, block, 0, st, pdl, p, (int)vx, (int)vw);
     if (epi == ZL_GEMM_EPI_GELU_TANH_MUL)
         return launch(k_gemm_mma<T, TO, ZL_GEMM_EPI_GELU_TANH_MUL>, grid, block, 0, st, pdl, p, (int)vx, (int)vw);
     if (epi == ZL_GEMM_EPI_SOFTCAP)
@@ -552,7 +554,7 @@ static int gemm_dispatch(GemmP p, int batch, int in_dtype, int out_dtype, int ep
     ZL_CHECK_ARG(p.ldx >= K && p.ldw >= K && p.ldy >= (pairs ? N / 2 : N));
     ZL_CHECK_ARG(in_dtype == ZL_F16 || in_dtype == ZL_BF16 || in_dtype == ZL_F32);
     ZL_CHECK_ARG(out_dtype == in_dtype || out_dtype == ZL_F32);
-    ZL_CHECK_ARG(epilogue >= ZL_GEMM_EPI_NONE && epilogue <= ZL_GEMM_EPI_SOFTCAP);
+    ZL_CHECK_ARG(epilogue >= ZL_GEMM_EPI_NONE && epilogue <= ZL_GEMM_EPI_REGLU);
     const bool gated = epilogue == ZL_GEMM_EPI_SIGMOID_GATE || epilogue == ZL_GEMM_EPI_GELU_TANH_MUL;
     ZL_CHECK_ARG(!gated || (p.gate && p.ldg >= N && !grouped));
     ZL_CHECK_ARG(epilogue != ZL_GEMM_EPI_SOFTCAP || p.limit > 0.f);
@@ -575,6 +577,8 @@ static int gemm_dispatch(GemmP p, int batch, int in_dtype, int out_dtype, int ep
             e = launch(k_gemm_f32<ZL_GEMM_EPI_GLU_CLAMP>, grid, block, 0, stream, pdl != 0, p, (int)vx, (int)vw);
         else if (epilogue == ZL_GEMM_EPI_GEGLU_TANH)
             e = launch(k_gemm_f32<ZL_GEMM_EPI_GEGLU_TANH>, grid, block, 0, stream, pdl != 0, p, (int)vx, (int)vw);
+        else if (epilogue == ZL_GEMM_EPI_REGLU)
+            e = launch(k_gemm_f32<ZL_GEMM_EPI_REGLU>, grid, block, 0, stream, pdl != 0, p, (int)vx, (int)vw);
         else if (epilogue == ZL_GEMM_EPI_GELU_TANH_MUL)
             e = launch(k_gemm_f32<ZL_GEMM_EPI_GELU_TANH_MUL>, grid, block, 0, stream, pdl != 0, p, (int)vx, (int)vw);
         else if (epilogue == ZL_GEMM_EPI_SOFTCAP)
@@ -592,7 +596,7 @@ static int gemm_dispatch(GemmP p, int batch, int in_dtype, int out_dtype, int ep
                                     : launch_grouped_small<__half, __half>(p, batch, pairs, pdl != 0, stream);
     } else if (!grouped && pairs && batch == 1 && M <= 8 && vx && vw && K % 8 == 0 &&
                (size_t)8 * K * 2 <= 160 * 1024) {   // a dense gated feed-forward of a decode step: gate and up rows streamed together
-        p.pair_gelu = epilogue == ZL_GEMM_EPI_GEGLU_TANH;
+        p.pair_fn = epilogue;
         if (in_dtype == ZL_BF16)
             e = out_dtype == ZL_F32 ? launch_grouped_small<__nv_bfloat16, float>(p, 1, true, pdl != 0, stream)
                                     : launch_grouped_small<__nv_bfloat16, __nv_bfloat16>(p, 1, true, pdl != 0, stream);

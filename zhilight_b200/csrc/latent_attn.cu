@@ -11,6 +11,11 @@
 //
 // Token t of a step sees the rows 0 .. pos[t] of its slot; the step's own latents are appended before this kernel, so
 // one kernel serves prompt portions (consecutive positions of one slot) and decode batches (one token per slot).
+//
+// General form (zl_latent_attention_ex): a cached row may carry more columns than the value has -- a rotated key part
+// shared by the heads behind the latent -- that enter the score only; the sink may be absent (an ordinary softmax); a
+// sigmoid gate per head may multiply the output; and the probabilities may enter the 16-bit product as a hi + lo pair,
+// so that no weight is rounded to 8 bits.  k_latent_rope_append writes such rows and the queries' rotated parts.
 #include "common.cuh"
 
 #include <math.h>
@@ -28,20 +33,27 @@ struct LaParams {
     void* const* slot_addrs;
     const int32_t* slot;
     const int32_t* pos;
-    const float* sink;     // (H)
+    const float* sink;     // (H) or null: no extra term
     void* out;             // (T, H, R) activation dtype
     float* part_acc;       // (T, H, S, R)
     float* part_ml;        // (T, H, S, 2)
     float scale;
     int H, R, HG, S;
+    int RS;                // columns of a cached row and of qa: the score runs over all of them, the value is the first R
+    const float* gate = nullptr;   // gate[t * ldg + h] logits or null
+    long long ldg = 0;
 };
+
+__device__ __forceinline__ float la_gate(const float* gate, long long ldg, int t, int h) {
+    return gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h])) : 1.0f;
+}
 
 template <typename TC, int EPT>
 __global__ void __launch_bounds__(kLaThreads) k_latent_attn(LaParams<TC> p) {
     extern __shared__ float smem[];
-    const int R = p.R, RP = R + 1;
-    float* sq = smem;                       // [HG][R]
-    float* sc = sq + p.HG * R;              // [32][R + 1]
+    const int R = p.R, RS = p.RS, RP = RS + 1;
+    float* sq = smem;                       // [HG][RS]
+    float* sc = sq + p.HG * RS;             // [32][RS + 1]
     float* sp = sc + kLaKeys * RP;          // [HG][32]
     float* sm = sp + p.HG * kLaKeys;        // [HG] running max
     float* sl = sm + p.HG;                  // [HG] running sum
@@ -59,10 +71,10 @@ __global__ void __launch_bounds__(kLaThreads) k_latent_attn(LaParams<TC> p) {
         lo = split * per;
         hi = min(len, lo + per);
     }
-    for (int i = tid; i < hg * R; i += kLaThreads) sq[i] = p.qa[((size_t)t * p.H + h0) * R + i];
-    if (tid < hg) {
-        sm[tid] = p.S > 1 ? -INFINITY : p.sink[h0 + tid];
-        sl[tid] = p.S > 1 ? 0.f : 1.f;
+    for (int i = tid; i < hg * RS; i += kLaThreads) sq[i] = p.qa[((size_t)t * p.H + h0) * RS + i];
+    for (int i = tid; i < hg; i += kLaThreads) {
+        sm[i] = p.S > 1 || !p.sink ? -INFINITY : p.sink[h0 + i];
+        sl[i] = p.S > 1 || !p.sink ? 0.f : 1.f;
     }
     float acc[EPT];
 #pragma unroll
@@ -70,16 +82,16 @@ __global__ void __launch_bounds__(kLaThreads) k_latent_attn(LaParams<TC> p) {
 
     for (int j0 = lo; j0 < hi; j0 += kLaKeys) {
         __syncthreads();   // previous tile fully consumed (and sq / sm / sl initialised)
-        for (int i = tid; i < kLaKeys * R; i += kLaThreads) {
-            const int j = i / R, r = i - j * R;
-            sc[j * RP + r] = (j0 + j < hi) ? to_f32<TC>(cache[(size_t)(j0 + j) * R + r]) : 0.f;
+        for (int i = tid; i < kLaKeys * RS; i += kLaThreads) {
+            const int j = i / RS, r = i - j * RS;
+            sc[j * RP + r] = (j0 + j < hi) ? to_f32<TC>(cache[(size_t)(j0 + j) * RS + r]) : 0.f;
         }
         __syncthreads();
         for (int hh = warp; hh < hg; hh += kLaThreads / 32) {
-            const float* q = sq + hh * R;
+            const float* q = sq + hh * RS;
             const float* c = sc + lane * RP;
             float s = 0.f;
-            for (int r = 0; r < R; ++r) s = fmaf(q[r], c[r], s);
+            for (int r = 0; r < RS; ++r) s = fmaf(q[r], c[r], s);
             const bool valid = j0 + lane < hi;
             s = valid ? s * p.scale : -INFINITY;
             const float m_old = sm[hh];
@@ -117,20 +129,21 @@ __global__ void __launch_bounds__(kLaThreads) k_latent_attn(LaParams<TC> p) {
             const int hh = e / R, r = e - hh * R;
             const size_t th = (size_t)t * p.H + h0 + hh;
             if (p.S > 1) p.part_acc[(th * p.S + split) * R + r] = acc[k];
-            else static_cast<TC*>(p.out)[th * R + r] = from_f32<TC>(acc[k] / sl[hh]);
+            else static_cast<TC*>(p.out)[th * R + r] = from_f32<TC>(acc[k] / sl[hh] * la_gate(p.gate, p.ldg, t, h0 + hh));
         }
     }
-    if (p.S > 1 && tid < hg) {
-        const size_t th = (size_t)t * p.H + h0 + tid;
-        p.part_ml[(th * p.S + split) * 2 + 0] = sm[tid];
-        p.part_ml[(th * p.S + split) * 2 + 1] = sl[tid];
+    for (int i = tid; p.S > 1 && i < hg; i += kLaThreads) {
+        const size_t th = (size_t)t * p.H + h0 + i;
+        p.part_ml[(th * p.S + split) * 2 + 0] = sm[i];
+        p.part_ml[(th * p.S + split) * 2 + 1] = sl[i];
     }
 }
 
 // grid (H, T): merge the S <= 64 partial (max, sum, accumulator) triples of one (token, head) and the sink
 template <typename TC>
 __global__ void k_latent_attn_merge(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                    const float* __restrict__ sink, TC* __restrict__ out, int H, int R, int S) {
+                                    const float* __restrict__ sink, const float* __restrict__ gate, long long ldg,
+                                    TC* __restrict__ out, int H, int R, int S) {
     __shared__ float wgt[64];
     pdl_trigger();
     pdl_wait();
@@ -138,14 +151,15 @@ __global__ void k_latent_attn_merge(const float* __restrict__ part_acc, const fl
     if (threadIdx.x < 32) {
         const int lane = threadIdx.x;
         const float* ml = part_ml + th * S * 2;
-        const float sk = sink[blockIdx.x];
+        const float sk = sink ? sink[blockIdx.x] : -INFINITY;
         const float m0 = lane < S ? ml[2 * lane] : -INFINITY, m1 = lane + 32 < S ? ml[2 * (lane + 32)] : -INFINITY;
         const float l0 = lane < S ? ml[2 * lane + 1] : 0.f, l1 = lane + 32 < S ? ml[2 * (lane + 32) + 1] : 0.f;
         const float M = fmaxf(sk, warp_max(fmaxf(m0, m1)));
         const float e0 = m0 == -INFINITY ? 0.f : expf(m0 - M), e1 = m1 == -INFINITY ? 0.f : expf(m1 - M);
         const float L = expf(sk - M) + warp_sum(l0 * e0 + l1 * e1);
-        wgt[lane] = e0 / L;
-        wgt[lane + 32] = e1 / L;
+        const float gl = la_gate(gate, ldg, blockIdx.y, blockIdx.x) / L;
+        wgt[lane] = e0 * gl;
+        wgt[lane + 32] = e1 * gl;
     }
     __syncthreads();
     const float* pa = part_acc + th * S * R;
@@ -183,9 +197,12 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* 
                  : "r"(smem_u32(smem_row)));
 }
 
-template <int NK>   // kv_rank = 64 * NK: every warp contracts over 16 * NK and owns 16 * NK output columns
+// NK: the value has 64 * NK columns, every warp contracts over 16 * NK of them and owns 16 * NK output columns.  EX: the
+// general form -- up to 64 score-only columns behind them (16 per warp), no sink, gate, probabilities as a hi + lo pair.
+template <int NK, bool EX>
 __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16> p) {
-    constexpr int RQ = 16 * NK, R = 4 * RQ, RP = R + 8;
+    constexpr int RQ = 16 * NK, R = 4 * RQ;
+    const int RS = EX ? p.RS : R, RP = RS + 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* sc = reinterpret_cast<__nv_bfloat16*>(smem_raw);                       // [stages][32][RP]
     float* ss = reinterpret_cast<float*>(smem_raw + (size_t)kLmStages * kLmKeys * RP * 2);   // [4][16][34]
@@ -205,23 +222,36 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
     // query fragments of this warp's contraction quarter
     uint32_t qf[NK][4];
     {
-        const float* qa = p.qa + ((size_t)t * p.H) * R + warp * RQ;
+        const float* qa = p.qa + ((size_t)t * p.H) * RS + warp * RQ;
 #pragma unroll
         for (int ks = 0; ks < NK; ++ks) {
             const int k = ks * 16 + 2 * q4;
             const float2 z = make_float2(0.f, 0.f);
-            const float2 a0 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * R + k) : z;
-            const float2 a1 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * R + k) : z;
-            const float2 a2 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * R + k + 8) : z;
-            const float2 a3 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * R + k + 8) : z;
+            const float2 a0 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * RS + k) : z;
+            const float2 a1 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * RS + k) : z;
+            const float2 a2 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * RS + k + 8) : z;
+            const float2 a3 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * RS + k + 8) : z;
             qf[ks][0] = pack_bf16(a0.x, a0.y), qf[ks][1] = pack_bf16(a1.x, a1.y);
             qf[ks][2] = pack_bf16(a2.x, a2.y), qf[ks][3] = pack_bf16(a3.x, a3.y);
         }
     }
+    const bool extra = EX && warp * 16 < RS - R;   // this warp's 16 score-only columns
+    uint32_t qx[4] = {0, 0, 0, 0};
+    if (extra) {
+        const float* qa = p.qa + ((size_t)t * p.H) * RS + R + warp * 16 + 2 * q4;
+        const float2 z = make_float2(0.f, 0.f);
+        const float2 a0 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * RS) : z;
+        const float2 a1 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * RS) : z;
+        const float2 a2 = ha < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)ha * RS + 8) : z;
+        const float2 a3 = hb < p.H ? *reinterpret_cast<const float2*>(qa + (size_t)hb * RS + 8) : z;
+        qx[0] = pack_bf16(a0.x, a0.y), qx[1] = pack_bf16(a1.x, a1.y);
+        qx[2] = pack_bf16(a2.x, a2.y), qx[3] = pack_bf16(a3.x, a3.y);
+    }
     float m_run[2], l_run[2];
-    m_run[0] = p.S > 1 ? -INFINITY : (ha < p.H ? p.sink[ha] : 0.f);
-    m_run[1] = p.S > 1 ? -INFINITY : (hb < p.H ? p.sink[hb] : 0.f);
-    l_run[0] = l_run[1] = p.S > 1 ? 0.f : 1.f;
+    const bool with_sink = p.S == 1 && (!EX || p.sink);
+    m_run[0] = !with_sink ? -INFINITY : (ha < p.H ? p.sink[ha] : 0.f);
+    m_run[1] = !with_sink ? -INFINITY : (hb < p.H ? p.sink[hb] : 0.f);
+    l_run[0] = l_run[1] = with_sink ? 1.f : 0.f;
     float o[2 * NK][4];
 #pragma unroll
     for (int i = 0; i < 2 * NK; ++i)
@@ -230,9 +260,9 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
 
     auto stage = [&](int j0, int buf) {   // 32 keys x R bf16 in 16-byte pieces; keys past `hi` are zero rows
         __nv_bfloat16* dst = sc + (size_t)buf * kLmKeys * RP;
-        for (int i = tid; i < kLmKeys * (R / 8); i += 128) {
-            const int j = i / (R / 8), c8 = (i - j * (R / 8)) * 8;
-            if (j0 + j < hi) cp_async16(dst + j * RP + c8, cache + (size_t)(j0 + j) * R + c8);
+        for (int i = tid; i < kLmKeys * (RS / 8); i += 128) {
+            const int j = i / (RS / 8), c8 = (i - j * (RS / 8)) * 8;
+            if (j0 + j < hi) cp_async16(dst + j * RP + c8, cache + (size_t)(j0 + j) * RS + c8);
             else *reinterpret_cast<uint4*>(dst + j * RP + c8) = make_uint4(0, 0, 0, 0);
         }
         cp_async_commit();
@@ -260,6 +290,12 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
                 const uint32_t b0 = *reinterpret_cast<const uint32_t*>(krow + ks * 16);
                 const uint32_t b1 = *reinterpret_cast<const uint32_t*>(krow + ks * 16 + 8);
                 mma_16816_bf16(s[nt], qf[ks], b0, b1, s[nt]);
+            }
+            if (extra) {
+                const __nv_bfloat16* xrow = ct + (nt * 8 + g) * RP + R + warp * 16 + 2 * q4;
+                const uint32_t b0 = *reinterpret_cast<const uint32_t*>(xrow);
+                const uint32_t b1 = *reinterpret_cast<const uint32_t*>(xrow + 8);
+                mma_16816_bf16(s[nt], qx, b0, b1, s[nt]);
             }
         }
         float* mine = ss + warp * (kLmRows * 34);
@@ -298,7 +334,7 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
             m_run[r] = m_new;
             mx[r] = m_use;
         }
-        uint32_t pf[2][4];
+        uint32_t pf[2][4], pl[2][4];
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
             const float p0 = expf(s[nt][0] - mx[0]), p1 = expf(s[nt][1] - mx[0]);
@@ -307,6 +343,11 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
             sum[1] += p2 + p3;
             pf[nt >> 1][(nt & 1) * 2 + 0] = pack_bf16(p0, p1);
             pf[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16(p2, p3);
+            if constexpr (EX) {
+                auto lo = [](float v) { return v - __bfloat162float(__float2bfloat16_rn(v)); };
+                pl[nt >> 1][(nt & 1) * 2 + 0] = pack_bf16(lo(p0), lo(p1));
+                pl[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16(lo(p2), lo(p3));
+            }
         }
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
@@ -322,9 +363,18 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
             ldmatrix_x4_trans(bv, ct + lane * RP + warp * RQ + nt * 8);
             mma_16816_bf16(o[nt], pf[0], bv[0], bv[1], o[nt]);
             mma_16816_bf16(o[nt], pf[1], bv[2], bv[3], o[nt]);
+            if constexpr (EX) {
+                mma_16816_bf16(o[nt], pl[0], bv[0], bv[1], o[nt]);
+                mma_16816_bf16(o[nt], pl[1], bv[2], bv[3], o[nt]);
+            }
         }
     }
     const size_t tha = (size_t)t * p.H + ha, thb = (size_t)t * p.H + hb;
+    float fa = 1.0f / l_run[0], fb = 1.0f / l_run[1];
+    if (EX && p.S == 1 && p.gate) {
+        if (ha < p.H) fa *= la_gate(p.gate, p.ldg, t, ha);
+        if (hb < p.H) fb *= la_gate(p.gate, p.ldg, t, hb);
+    }
 #pragma unroll
     for (int nt = 0; nt < 2 * NK; ++nt) {
         const int col = warp * RQ + nt * 8 + 2 * q4;
@@ -334,9 +384,9 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
         } else {
             __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
             if (ha < p.H)
-                *reinterpret_cast<uint32_t*>(out + tha * R + col) = pack_bf16(o[nt][0] / l_run[0], o[nt][1] / l_run[0]);
+                *reinterpret_cast<uint32_t*>(out + tha * R + col) = pack_bf16(o[nt][0] * fa, o[nt][1] * fa);
             if (hb < p.H)
-                *reinterpret_cast<uint32_t*>(out + thb * R + col) = pack_bf16(o[nt][2] / l_run[1], o[nt][3] / l_run[1]);
+                *reinterpret_cast<uint32_t*>(out + thb * R + col) = pack_bf16(o[nt][2] * fb, o[nt][3] * fb);
         }
     }
     if (p.S > 1 && warp == 0 && q4 == 0) {
@@ -349,24 +399,52 @@ static bool lm_eligible(int dtype, int R) {
     static const bool off = getenv("ZL_LATENT_ATTN_NO_MMA") != nullptr;
     return !off && dtype == ZL_BF16 && R % 64 == 0 && R >= 64 && R <= 512;
 }
-static size_t lm_smem_bytes(int R) { return (size_t)kLmStages * kLmKeys * (R + 8) * 2 + (size_t)4 * kLmRows * 34 * 4; }
+static size_t lm_smem_bytes(int RS) { return (size_t)kLmStages * kLmKeys * (RS + 8) * 2 + (size_t)4 * kLmRows * 34 * 4; }
+// the general form needs its score-only columns in whole 16-column steps, at most one per warp
+static bool lm_eligible_ex(int dtype, int R, int RS) {
+    return lm_eligible(dtype, R) && (RS - R) % 16 == 0 && RS - R <= 64 && lm_smem_bytes(RS) <= 200 * 1024;
+}
 
+template <int NK, bool EX>
+static cudaError_t lm_attr(int bytes) {   // the largest request stands: models of several sizes may live side by side
+    static int set_for = 0;
+    if (bytes <= 48 * 1024 || bytes <= set_for) return cudaSuccess;
+    const cudaError_t e = cudaFuncSetAttribute(k_latent_attn_mma<NK, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e == cudaSuccess) set_for = bytes;
+    return e;
+}
+template <bool EX>
+static cudaError_t lm_prepare(int R, int RS) {
+    const int b = (int)lm_smem_bytes(RS);
+    switch (R / 64) {
+        case 1: return lm_attr<1, EX>(b);
+        case 2: return lm_attr<2, EX>(b);
+        case 3: return lm_attr<3, EX>(b);
+        case 4: return lm_attr<4, EX>(b);
+        case 5: return lm_attr<5, EX>(b);
+        case 6: return lm_attr<6, EX>(b);
+        case 7: return lm_attr<7, EX>(b);
+        default: return lm_attr<8, EX>(b);
+    }
+}
+
+template <bool EX>
 static int lm_launch(const LaParams<__nv_bfloat16>& p, int T, bool pdl, cudaStream_t st) {
-    const size_t smem = lm_smem_bytes(p.R);
+    const size_t smem = lm_smem_bytes(p.RS);
     const dim3 grid(cdiv(p.H, kLmRows), T, p.S), block(128);
     switch (p.R / 64) {
-        case 1: ZL_CHECK_CUDA(launch(k_latent_attn_mma<1>, grid, block, smem, st, pdl, p)); break;
-        case 2: ZL_CHECK_CUDA(launch(k_latent_attn_mma<2>, grid, block, smem, st, pdl, p)); break;
-        case 3: ZL_CHECK_CUDA(launch(k_latent_attn_mma<3>, grid, block, smem, st, pdl, p)); break;
-        case 4: ZL_CHECK_CUDA(launch(k_latent_attn_mma<4>, grid, block, smem, st, pdl, p)); break;
-        case 5: ZL_CHECK_CUDA(launch(k_latent_attn_mma<5>, grid, block, smem, st, pdl, p)); break;
-        case 6: ZL_CHECK_CUDA(launch(k_latent_attn_mma<6>, grid, block, smem, st, pdl, p)); break;
-        case 7: ZL_CHECK_CUDA(launch(k_latent_attn_mma<7>, grid, block, smem, st, pdl, p)); break;
-        default: ZL_CHECK_CUDA(launch(k_latent_attn_mma<8>, grid, block, smem, st, pdl, p)); break;
+        case 1: ZL_CHECK_CUDA(launch(k_latent_attn_mma<1, EX>, grid, block, smem, st, pdl, p)); break;
+        case 2: ZL_CHECK_CUDA(launch(k_latent_attn_mma<2, EX>, grid, block, smem, st, pdl, p)); break;
+        case 3: ZL_CHECK_CUDA(launch(k_latent_attn_mma<3, EX>, grid, block, smem, st, pdl, p)); break;
+        case 4: ZL_CHECK_CUDA(launch(k_latent_attn_mma<4, EX>, grid, block, smem, st, pdl, p)); break;
+        case 5: ZL_CHECK_CUDA(launch(k_latent_attn_mma<5, EX>, grid, block, smem, st, pdl, p)); break;
+        case 6: ZL_CHECK_CUDA(launch(k_latent_attn_mma<6, EX>, grid, block, smem, st, pdl, p)); break;
+        case 7: ZL_CHECK_CUDA(launch(k_latent_attn_mma<7, EX>, grid, block, smem, st, pdl, p)); break;
+        default: ZL_CHECK_CUDA(launch(k_latent_attn_mma<8, EX>, grid, block, smem, st, pdl, p)); break;
     }
     if (p.S > 1)
         ZL_CHECK_CUDA(launch(k_latent_attn_merge<__nv_bfloat16>, dim3(p.H, T), dim3(128), 0, st, pdl, (const float*)p.part_acc,
-                             (const float*)p.part_ml, p.sink, static_cast<__nv_bfloat16*>(p.out), p.H, p.R, p.S));
+                             (const float*)p.part_ml, p.sink, p.gate, p.ldg, static_cast<__nv_bfloat16*>(p.out), p.H, p.R, p.S));
     return ZL_OK;
 }
 
@@ -375,13 +453,13 @@ static int la_heads_per_cta(int H, int R) {
     if (hg < 1) hg = 1;
     return hg < H ? hg : H;
 }
-static size_t la_smem_bytes(int HG, int R) {
-    return sizeof(float) * ((size_t)HG * R + (size_t)kLaKeys * (R + 1) + (size_t)HG * kLaKeys + 3 * (size_t)HG);
+static size_t la_smem_bytes(int HG, int RS) {
+    return sizeof(float) * ((size_t)HG * RS + (size_t)kLaKeys * (RS + 1) + (size_t)HG * kLaKeys + 3 * (size_t)HG);
 }
 
 template <typename TC>
 static int la_launch(LaParams<TC> p, int T, bool pdl, cudaStream_t st) {
-    const size_t smem = la_smem_bytes(p.HG, p.R);
+    const size_t smem = la_smem_bytes(p.HG, p.RS);
     const int ept = cdiv(p.HG * p.R, kLaThreads);
     const dim3 grid(T, cdiv(p.H, p.HG), p.S), block(kLaThreads);
 #define ZL_LA_CASE(E)                                                                                        \
@@ -395,8 +473,61 @@ static int la_launch(LaParams<TC> p, int T, bool pdl, cudaStream_t st) {
 #undef ZL_LA_CASE
     if (p.S > 1)
         ZL_CHECK_CUDA(launch(k_latent_attn_merge<TC>, dim3(p.H, T), dim3(128), 0, st, pdl, (const float*)p.part_acc,
-                             (const float*)p.part_ml, p.sink, static_cast<TC*>(p.out), p.H, p.R, p.S));
+                             (const float*)p.part_ml, p.sink, p.gate, p.ldg, static_cast<TC*>(p.out), p.H, p.R, p.S));
     return ZL_OK;
+}
+
+// one warp per (token, unit): the H query heads, then the rotated key part, then the latent (norm and append)
+struct LaPrepP {
+    const float* proj;
+    long long ldp;
+    int q_off, H, d, rd;
+    const float2* table;       // (T, rd / 2)
+    void* q_out;
+    float* qa;
+    int c_off, R;
+    const float* kv_w;
+    int rank_cols, row_cols;
+    void* const* slot_addrs;
+    const int32_t *slot, *pos;
+    float eps;
+};
+template <typename TO>
+__global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.y, unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit > p.H + 1) return;
+    const float* row = p.proj + (size_t)t * p.ldp;
+    const float2* tab = p.table + (size_t)t * (p.rd >> 1);
+    if (unit < p.H) {
+        const float* src = row + p.q_off + (size_t)unit * (p.d + p.rd);
+        TO* dst = static_cast<TO*>(p.q_out) + ((size_t)t * p.H + unit) * p.d;
+        for (int c = lane; c < p.d; c += 32) dst[c] = from_f32<TO>(src[c]);
+        float* qr = p.qa + ((size_t)t * p.H + unit) * p.row_cols + p.rank_cols;
+        for (int i = lane; i < (p.rd >> 1); i += 32) {
+            const float u = src[p.d + 2 * i], v = src[p.d + 2 * i + 1];
+            const float2 cs = tab[i];
+            qr[2 * i] = u * cs.x - v * cs.y;
+            qr[2 * i + 1] = v * cs.x + u * cs.y;
+        }
+        return;
+    }
+    TO* dst = static_cast<TO*>(p.slot_addrs[p.slot[t]]) + (size_t)p.pos[t] * p.row_cols;
+    const float* src = row + p.c_off;
+    if (unit == p.H) {
+        for (int i = lane; i < (p.rd >> 1); i += 32) {
+            const float u = src[p.R + 2 * i], v = src[p.R + 2 * i + 1];
+            const float2 cs = tab[i];
+            dst[p.rank_cols + 2 * i] = from_f32<TO>(u * cs.x - v * cs.y);
+            dst[p.rank_cols + 2 * i + 1] = from_f32<TO>(v * cs.x + u * cs.y);
+        }
+        return;
+    }
+    float ss = 0.f;
+    for (int c = lane; c < p.R; c += 32) ss = fmaf(src[c], src[c], ss);
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)p.R + p.eps);
+    for (int c = lane; c < p.R; c += 32) dst[c] = from_f32<TO>(src[c] * r * p.kv_w[c]);
 }
 
 }  // namespace zl
@@ -410,10 +541,13 @@ extern "C" size_t zl_latent_attention_workspace_bytes(int T, int heads, int kv_r
 
 template <typename TC>
 static int la_prepare(size_t smem) {
+    static size_t set_for = 0;
+    if (smem <= 48 * 1024 || smem <= set_for) return ZL_OK;
     ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn<TC, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn<TC, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn<TC, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn<TC, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    set_for = smem;
     return ZL_OK;
 }
 
@@ -431,45 +565,80 @@ extern "C" int zl_latent_attention_splits(int T, int heads, int kv_rank, int max
 
 // opt-in shared memory of the kernel for this shape; call once outside any stream capture
 extern "C" int zl_latent_attention_prepare(int heads, int kv_rank, int dtype) {
-    ZL_CHECK_ARG(heads > 0 && kv_rank > 0);
-    ZL_CHECK_SUPPORTED(kv_rank <= kLaMaxElems);
-    const size_t smem = la_smem_bytes(la_heads_per_cta(heads, kv_rank), kv_rank);
+    if (lm_eligible(dtype, kv_rank)) ZL_CHECK_CUDA(lm_prepare<false>(kv_rank, kv_rank));
+    return zl_latent_attention_prepare_ex(heads, kv_rank, kv_rank, dtype);
+}
+
+extern "C" int zl_latent_attention_prepare_ex(int heads, int rank_cols, int row_cols, int dtype) {
+    ZL_CHECK_ARG(heads > 0 && rank_cols > 0 && row_cols >= rank_cols);
+    ZL_CHECK_ARG(dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32);
+    ZL_CHECK_SUPPORTED(rank_cols <= kLaMaxElems);
+    const size_t smem = la_smem_bytes(la_heads_per_cta(heads, rank_cols), row_cols);
     ZL_CHECK_SUPPORTED(smem <= 200 * 1024);
-    if (lm_eligible(dtype, kv_rank) && lm_smem_bytes(kv_rank) > 48 * 1024) {
-        const int b = (int)lm_smem_bytes(kv_rank);
-        ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn_mma<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, b));
-        ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn_mma<5>, cudaFuncAttributeMaxDynamicSharedMemorySize, b));
-        ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn_mma<6>, cudaFuncAttributeMaxDynamicSharedMemorySize, b));
-        ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn_mma<7>, cudaFuncAttributeMaxDynamicSharedMemorySize, b));
-        ZL_CHECK_CUDA(cudaFuncSetAttribute(k_latent_attn_mma<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, b));
-    }
-    if (smem <= 48 * 1024) return ZL_OK;
+    if (lm_eligible_ex(dtype, rank_cols, row_cols)) ZL_CHECK_CUDA(lm_prepare<true>(rank_cols, row_cols));
     if (dtype == ZL_F32) return la_prepare<float>(smem);
     if (dtype == ZL_BF16) return la_prepare<__nv_bfloat16>(smem);
     return la_prepare<__half>(smem);
+}
+
+template <typename TC>
+static LaParams<TC> la_params(const float* qa, void* const* slot_addrs, const int32_t* slot, const int32_t* pos, const float* sink,
+                              float scale, void* out, int T, int heads, int R, int RS, int splits, void* workspace,
+                              const float* gate, long long ldg) {
+    float* part_acc = static_cast<float*>(workspace);
+    float* part_ml = splits > 1 ? part_acc + (size_t)T * heads * splits * R : nullptr;
+    return LaParams<TC>{qa, slot_addrs, slot, pos, sink, out, part_acc, part_ml, scale, heads, R, la_heads_per_cta(heads, R), splits,
+                        RS, gate, ldg};
 }
 
 extern "C" int zl_latent_attention(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
                                    const float* sink, float scale, void* out, int T, int heads, int kv_rank, int splits,
                                    void* workspace, size_t workspace_bytes, int dtype, int pdl, zl_stream_t stream) {
     ZL_CHECK_ARG(q_absorbed && slot_addrs && slot && pos && sink && out && T > 0 && heads > 0 && kv_rank > 0);
-    ZL_CHECK_ARG(dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32);
     ZL_CHECK_ARG(splits >= 1 && splits <= 65535 && heads <= 65535);
     ZL_CHECK_SUPPORTED(kv_rank <= kLaMaxElems);
     ZL_CHECK_ARG(workspace_bytes >= zl_latent_attention_workspace_bytes(T, heads, kv_rank, splits) && (splits == 1 || workspace));
-    const int HG = la_heads_per_cta(heads, kv_rank);
-    ZL_CHECK_SUPPORTED(la_smem_bytes(HG, kv_rank) <= 200 * 1024);
-    float* part_acc = static_cast<float*>(workspace);
-    float* part_ml = splits > 1 ? part_acc + (size_t)T * heads * splits * kv_rank : nullptr;
-    if (dtype == ZL_F32) {
-        LaParams<float> p{q_absorbed, slot_addrs, slot, pos, sink, out, part_acc, part_ml, scale, heads, kv_rank, HG, splits};
-        return la_launch<float>(p, T, pdl != 0, stream);
-    }
-    if (dtype == ZL_BF16) {
-        LaParams<__nv_bfloat16> p{q_absorbed, slot_addrs, slot, pos, sink, out, part_acc, part_ml, scale, heads, kv_rank, HG, splits};
-        if (lm_eligible(dtype, kv_rank) && (reinterpret_cast<uintptr_t>(q_absorbed) & 7) == 0) return lm_launch(p, T, pdl != 0, stream);
-        return la_launch<__nv_bfloat16>(p, T, pdl != 0, stream);
-    }
-    LaParams<__half> p{q_absorbed, slot_addrs, slot, pos, sink, out, part_acc, part_ml, scale, heads, kv_rank, HG, splits};
-    return la_launch<__half>(p, T, pdl != 0, stream);
+    if (lm_eligible(dtype, kv_rank) && (reinterpret_cast<uintptr_t>(q_absorbed) & 7) == 0)
+        return lm_launch<false>(la_params<__nv_bfloat16>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, kv_rank, kv_rank,
+                                                         splits, workspace, nullptr, 0), T, pdl != 0, stream);
+    return zl_latent_attention_ex(q_absorbed, slot_addrs, slot, pos, sink, nullptr, 0, scale, out, T, heads, kv_rank, kv_rank, splits,
+                                  workspace, workspace_bytes, dtype, pdl, stream);
+}
+
+extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                                      const float* sink, const float* gate, long long ldg, float scale, void* out, int T,
+                                      int heads, int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
+                                      int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(q_absorbed && slot_addrs && slot && pos && out && T > 0 && T <= 65535 && heads > 0 && rank_cols > 0);
+    ZL_CHECK_ARG(row_cols >= rank_cols && (dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32));
+    ZL_CHECK_ARG(splits >= 1 && splits <= 64 && heads <= 65535);
+    ZL_CHECK_SUPPORTED(rank_cols <= kLaMaxElems);
+    ZL_CHECK_ARG(workspace_bytes >= zl_latent_attention_workspace_bytes(T, heads, rank_cols, splits) && (splits == 1 || workspace));
+    ZL_CHECK_SUPPORTED(la_smem_bytes(la_heads_per_cta(heads, rank_cols), row_cols) <= 200 * 1024);
+#define ZL_LA_P(TC) \
+    la_params<TC>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, rank_cols, row_cols, splits, workspace, gate, ldg)
+    if (dtype == ZL_F32) return la_launch<float>(ZL_LA_P(float), T, pdl != 0, stream);
+    if (dtype == ZL_F16) return la_launch<__half>(ZL_LA_P(__half), T, pdl != 0, stream);
+    if (lm_eligible_ex(dtype, rank_cols, row_cols) && row_cols % 8 == 0 && (reinterpret_cast<uintptr_t>(q_absorbed) & 7) == 0)
+        return lm_launch<true>(ZL_LA_P(__nv_bfloat16), T, pdl != 0, stream);
+    return la_launch<__nv_bfloat16>(ZL_LA_P(__nv_bfloat16), T, pdl != 0, stream);
+#undef ZL_LA_P
+}
+
+extern "C" int zl_latent_rope_append(const float* proj, long long ldp, int q_off, int heads, int dim, int rot_dim,
+                                     const float* table, void* q_out, float* qa, int c_off, int kv_rank, const float* kv_weight,
+                                     int rank_cols, int row_cols, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                                     int T, float eps, int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(proj && q_out && qa && kv_weight && slot_addrs && slot && pos && T > 0 && T <= 65535 && heads > 0 && dim > 0);
+    ZL_CHECK_ARG(kv_rank > 0 && rank_cols >= kv_rank && rot_dim >= 0 && rot_dim % 2 == 0 && row_cols >= rank_cols + rot_dim);
+    ZL_CHECK_ARG((rot_dim == 0 || table) && (dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32));
+    const LaPrepP p{proj, ldp, q_off, heads, dim, rot_dim, reinterpret_cast<const float2*>(table), q_out, qa, c_off, kv_rank, kv_weight,
+                    rank_cols, row_cols, slot_addrs, slot, pos, eps};
+    const dim3 grid(cdiv(heads + 2, 8), T), block(256);
+    cudaError_t e;
+    if (dtype == ZL_F32) e = launch(k_latent_rope_append<float>, grid, block, 0, stream, pdl != 0, p);
+    else if (dtype == ZL_BF16) e = launch(k_latent_rope_append<__nv_bfloat16>, grid, block, 0, stream, pdl != 0, p);
+    else e = launch(k_latent_rope_append<__half>, grid, block, 0, stream, pdl != 0, p);
+    ZL_CHECK_CUDA(e);
+    return ZL_OK;
 }

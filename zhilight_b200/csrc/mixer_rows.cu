@@ -15,7 +15,10 @@
 //   * rotations from a per-step (cos, sin) table: queries and keys over their first rot_dims dimensions and values over
 //     all of theirs, pairs in halves or adjacent, no norms, with the append to the slot's caches;
 //   * the residual update of a parallel layer: both sublayers' results times a layer scale and a sigmoid gate per channel,
-//     the second a weighted sum of parts of which some may be the sublayers' input itself, then the next layer's norm.
+//     the second a weighted sum of parts of which some may be the sublayers' input itself, then the next layer's norm;
+//   * the residual update of a pre-norm layer: x += a weighted sum of parts, then the next sublayer's norm and / or a copy of
+//     the new x in the activation dtype;
+//   * the embedding row as the start of the stream, with the same two outputs.
 #include "common.cuh"
 
 #include <cmath>
@@ -576,9 +579,156 @@ __global__ void __launch_bounds__(256) k_gated_parallel_combine(GatedCombineP p,
     for (int c = threadIdx.x; c < D; c += 256) h[c] = from_f32<TO>(gsx[c] * r * p.next_w[c]);
 }
 
+struct ResidualNormP {
+    float* x;
+    long long ldx;
+    const float* parts;        // n_parts rows per token, or null: x is the input as it is
+    long long ldp;
+    const float* coef;         // (T, n_parts) or null: ones
+    int n_parts;
+    const int32_t* ids;        // embedding form: x[t] = table[ids[t]] (no parts)
+    const void* table;
+    int vocab;
+    const float* next_w;       // multipliers of the next norm, or null
+    void* h;                   // (T, D)
+    void* copy1;               // the new x in the activation dtype, or null
+    void* copy2;               // a second copy, or null
+    long long ldc;             // row stride of the copies
+    int D;
+    float eps;
+};
+
+// One CTA per token.  vec (D % 4 == 0, D <= 4096, every row 16-byte aligned): a thread keeps its (up to four) 4-channel
+// pieces of the new x in registers between the sum and the norm; otherwise channel by channel through x itself.
+template <typename TO>
+__global__ void __launch_bounds__(256) k_residual_norm(ResidualNormP p, int vec) {
+    __shared__ float red[8];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, D = p.D;
+    float* xr = p.x + (size_t)t * p.ldx;
+    const float* pr = p.parts ? p.parts + (size_t)t * p.n_parts * p.ldp : nullptr;
+    const float* cf = p.coef ? p.coef + (size_t)t * p.n_parts : nullptr;
+    const TO* er = nullptr;
+    if (p.ids) {
+        const int id = p.ids[t];
+        er = static_cast<const TO*>(p.table) + (size_t)(id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id)) * D;
+    }
+    TO* h = p.next_w ? static_cast<TO*>(p.h) + (size_t)t * D : nullptr;
+    TO* c1 = p.copy1 ? static_cast<TO*>(p.copy1) + (size_t)t * p.ldc : nullptr;
+    TO* c2 = p.copy2 ? static_cast<TO*>(p.copy2) + (size_t)t * p.ldc : nullptr;
+    float ss = 0.f;
+    if (vec) {
+        float4 xv[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = (threadIdx.x + i * 256) * 4;
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c < D) {
+                if (er) s = make_float4(to_f32<TO>(er[c]), to_f32<TO>(er[c + 1]), to_f32<TO>(er[c + 2]), to_f32<TO>(er[c + 3]));
+                else s = ld4(xr + c);
+                if (pr) {
+                    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+                    for (int q = 0; q < p.n_parts; ++q) {
+                        const float w = cf ? cf[q] : 1.0f;
+                        const float4 v = ld4(pr + (size_t)q * p.ldp + c);
+                        f.x = fmaf(w, v.x, f.x), f.y = fmaf(w, v.y, f.y), f.z = fmaf(w, v.z, f.z), f.w = fmaf(w, v.w, f.w);
+                    }
+                    s.x += f.x, s.y += f.y, s.z += f.z, s.w += f.w;
+                }
+                if (pr || er) *reinterpret_cast<float4*>(xr + c) = s;
+                if (c1) store4<TO>(c1 + c, s.x, s.y, s.z, s.w);
+                if (c2) store4<TO>(c2 + c, s.x, s.y, s.z, s.w);
+            }
+            xv[i] = s;
+            ss = fmaf(s.x, s.x, fmaf(s.y, s.y, fmaf(s.z, s.z, fmaf(s.w, s.w, ss))));
+        }
+        if (!h) return;
+        const float r = 1.0f / sqrtf(block_sum_256(ss, red) / (float)D + p.eps);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = (threadIdx.x + i * 256) * 4;
+            if (c >= D) continue;
+            const float4 nw = ld4(p.next_w + c);
+            store4<TO>(h + c, xv[i].x * r * nw.x, xv[i].y * r * nw.y, xv[i].z * r * nw.z, xv[i].w * r * nw.w);
+        }
+        return;
+    }
+    for (int c = threadIdx.x; c < D; c += 256) {
+        float s = er ? to_f32<TO>(er[c]) : xr[c];
+        if (pr) {
+            float f = 0.f;
+            for (int q = 0; q < p.n_parts; ++q) f = fmaf(cf ? cf[q] : 1.0f, pr[(size_t)q * p.ldp + c], f);
+            s += f;
+        }
+        if (pr || er) xr[c] = s;
+        if (c1) c1[c] = from_f32<TO>(s);
+        if (c2) c2[c] = from_f32<TO>(s);
+        ss = fmaf(s, s, ss);
+    }
+    if (!h) return;
+    const float r = 1.0f / sqrtf(block_sum_256(ss, red) / (float)D + p.eps);
+    for (int c = threadIdx.x; c < D; c += 256) h[c] = from_f32<TO>(xr[c] * r * p.next_w[c]);   // a thread reads what it wrote
+}
+
 }  // namespace zl
 
 using namespace zl;
+
+static int residual_norm_launch(const ResidualNormP& p, int act_dtype, int T, int pdl, cudaStream_t stream) {
+    auto al = [](const void* q, int b) { return (reinterpret_cast<uintptr_t>(q) & (b - 1)) == 0; };
+    const int ab = act_dtype == ZL_F32 ? 16 : 8;   // store4 of the activation dtype
+    const int vec = p.D % 4 == 0 && p.D <= 4096 && p.ldx % 4 == 0 && al(p.x, 16) && (!p.parts || (p.ldp % 4 == 0 && al(p.parts, 16))) &&
+                    (!p.next_w || (al(p.next_w, 16) && al(p.h, ab))) &&
+                    (!(p.copy1 || p.copy2) || (p.ldc % 4 == 0 && al(p.copy1, ab) && al(p.copy2, ab)));
+    cudaError_t e;
+    if (act_dtype == ZL_F32) e = launch(k_residual_norm<float>, dim3(T), dim3(256), 0, stream, pdl != 0, p, vec);
+    else if (act_dtype == ZL_BF16) e = launch(k_residual_norm<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, pdl != 0, p, vec);
+    else e = launch(k_residual_norm<__half>, dim3(T), dim3(256), 0, stream, pdl != 0, p, vec);
+    ZL_CHECK_CUDA(e);
+    return ZL_OK;
+}
+
+extern "C" int zl_residual_norm(float* x, long long ldx, const float* parts, long long ldp, const float* coef, int n_parts,
+                                const float* next_w, void* h, void* x_copy, long long ld_copy, int act_dtype, int T, int D,
+                                float eps, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(x && T > 0 && D > 0 && ldx >= D && (!parts || (n_parts > 0 && ldp >= D)));
+    ZL_CHECK_ARG((!next_w || h) && (!x_copy || ld_copy >= D));
+    ZL_CHECK_ARG(act_dtype == ZL_F16 || act_dtype == ZL_BF16 || act_dtype == ZL_F32);
+    return residual_norm_launch(ResidualNormP{x, ldx, parts, ldp, coef, n_parts, nullptr, nullptr, 0, next_w, h, x_copy, nullptr,
+                                              ld_copy, D, eps}, act_dtype, T, pdl, stream);
+}
+
+extern "C" int zl_embed_norm(const int32_t* ids, const void* table, int vocab, float* x, const float* next_w, void* h,
+                             void* x_copy, void* x_copy2, long long ld_copy, int act_dtype, int T, int D, float eps, int pdl,
+                             zl_stream_t stream) {
+    ZL_CHECK_ARG(ids && table && vocab > 0 && x && T > 0 && D > 0);
+    ZL_CHECK_ARG((!next_w || h) && (!(x_copy || x_copy2) || ld_copy >= D));
+    ZL_CHECK_ARG(act_dtype == ZL_F16 || act_dtype == ZL_BF16 || act_dtype == ZL_F32);
+    return residual_norm_launch(ResidualNormP{x, D, nullptr, 0, nullptr, 0, ids, table, vocab, next_w, h, x_copy, x_copy2, ld_copy, D,
+                                              eps}, act_dtype, T, pdl, stream);
+}
+
+extern "C" int zl_rope_inv_freq_wavelength(double base, int dims, double factor, double low, double high, double original,
+                                           double* out) {
+    ZL_CHECK_ARG(base > 1.0 && dims >= 0 && dims % 2 == 0 && (dims == 0 || out));
+    ZL_CHECK_ARG(factor <= 0 || (original > 0 && low > 0 && high > 0));
+    const double kPi = 3.14159265358979323846;
+    for (int i = 0; i < dims / 2; ++i) {
+        double f = pow(base, -2.0 * i / dims);
+        if (factor > 0) {
+            const double wave = 2 * kPi / f;
+            if (wave > original / low) f = f / factor;
+            else if (wave >= original / high) {   // not shorter than original / high: blended
+                const double s = (original / wave - low) / (high - low);
+                f = (1 - s) * f / factor + s * f;
+            }
+        }
+        out[i] = f;
+    }
+    return ZL_OK;
+}
 
 extern "C" int zl_rope_table(const int32_t* pos, int T, const double* inv_freq, int half, float* table, int pdl,
                              zl_stream_t stream) {

@@ -7,6 +7,10 @@
 // gets dist_bias[h][min(pos - key, n_dist - 1)] added after the scale.  Two more options: no sink at all (an ordinary
 // softmax), and an output rotation: values that were cached turned by their own position give a sum that is turned back
 // by the query's position, pair by pair from a (cos, sin) table, in fp32 before the store.
+// With window > 0 a token sees only the last `window` keys up to its own.  Differential attention (MAPS = 2): a query
+// head has two maps, each with queries and keys of its own and its own softmax over the same values; the result is
+// a_1 - lambda a_2 over its root mean square, times a constant, optionally under a full-width sigmoid gate.  Both maps
+// of a head are computed by the same CTA (the values are read once) and meet in fp32 before the only store.
 //
 // k_sink_attn_mma (16-bit caches, head sizes that are multiples of 16, values up to 128 wide, at most 16 query heads per
 // key/value head): a CTA owns up to 64 rows = (consecutive tokens of one run) x (the query heads of one key/value
@@ -18,7 +22,7 @@
 // k_sink_attn: any head sizes up to 256 and any dtype; scores, softmax and the weighted sum in fp32 FMAs.  One CTA per
 // (token, query head); its 8 warps take the keys j = warp, warp + 8, ... (a fixed assignment: the result of a token
 // does not depend on the step it is computed in) with an online softmax each, merged in warp order with the sink term.
-#include "common.cuh"
+#include "sink_attn.cuh"
 
 #include <cmath>
 #include <cstdlib>
@@ -27,27 +31,6 @@
 namespace zl {
 
 constexpr int kSaWarps = 8, kSaMaxPerLane = 8;
-
-struct SinkAttnP {
-    const void* q;             // (T, H * d)
-    void* const* k_addrs;      // slot -> (max_seq, G, d)
-    void* const* v_addrs;      // slot -> (max_seq, G, vd)
-    const int32_t *slot, *pos;
-    const float* sink;         // (H) or null: sink 0
-    const float* gate;         // gate[t * ldg + h] logits or null
-    long long ldg;
-    void* out;                 // (T, H * vd)
-    int H, G, d, vd;
-    float scale;
-    int splits;
-    float* ws;                 // splits > 1: (T, H, splits, 2 + vd) partial (max, sum, weighted values)
-    int chunk = 0;             // > 0: keys below (pos / chunk) * chunk are not seen
-    const float* dist_bias = nullptr;   // (H, n_dist) added to the scaled score by distance, or null
-    int n_dist = 0;
-    int no_sink = 0;           // the denominator holds the keys only
-    const float* out_table = nullptr;   // (T, vd / 2) pairs (cos, sin): the output of token t is turned back by these angles
-    int out_layout = 0;        // ZL_ROT_HALVES: pair (m, m + vd / 2); ZL_ROT_ADJACENT: pair (2m, 2m + 1)
-};
 
 // the two channels of pair m
 __device__ __forceinline__ void sa_pair(const SinkAttnP& p, int m, int& c1, int& c2) {
@@ -61,26 +44,29 @@ __device__ __forceinline__ void sa_store_unrotated(T* out, int c1, int c2, float
     out[c2] = from_f32<T>((v * cs.x - u * cs.y) * mul);
 }
 
-// first key a token at `pos` sees
-__device__ __forceinline__ int sa_first_key(const SinkAttnP& p, int pos) { return p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0; }
+__device__ __forceinline__ float sa_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
 
-template <typename T>
+// MAPS = 2: warps 0 .. 3 compute the first map, 4 .. 7 the second
+template <typename T, int MAPS>
 __global__ void __launch_bounds__(kSaWarps * 32) k_sink_attn(SinkAttnP p) {
+    constexpr int WPM = kSaWarps / MAPS;    // warps per map
     extern __shared__ float ssm[];
-    float* sq = ssm;                        // d
-    float* sm_m = ssm + p.d;                // kSaWarps
+    float* sq = ssm;                        // MAPS * d
+    float* sm_m = ssm + MAPS * p.d;         // kSaWarps
     float* sm_l = sm_m + kSaWarps;          // kSaWarps
     float* sm_acc = sm_l + kSaWarps;        // kSaWarps * vd
     pdl_trigger();
     pdl_wait();
     const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = h / (p.H / p.G), pos = p.pos[t], sl = p.slot[t];
-    const T* q = static_cast<const T*>(p.q) + ((size_t)t * p.H + h) * p.d;
-    for (int c = threadIdx.x; c < p.d; c += blockDim.x) sq[c] = to_f32<T>(q[c]) * p.scale;
+    const int map = warp / WPM, wm = warp - map * WPM;
+    const T* q = static_cast<const T*>(p.q) + ((size_t)t * p.H + h) * MAPS * p.d;
+    for (int c = threadIdx.x; c < MAPS * p.d; c += blockDim.x) sq[c] = to_f32<T>(q[c]) * p.scale;
     __syncthreads();
-    const T* kc = static_cast<const T*>(p.k_addrs[sl]) + (size_t)g * p.d;
+    const T* kc = static_cast<const T*>(p.k_addrs[sl]) + ((size_t)g * MAPS + map) * p.d;
     const T* vc = static_cast<const T*>(p.v_addrs[sl]) + (size_t)g * p.vd;
-    const size_t kst = (size_t)p.G * p.d, vst = (size_t)p.G * p.vd;
+    const size_t kst = (size_t)p.G * MAPS * p.d, vst = (size_t)p.G * p.vd;
+    const float* sqm = sq + map * p.d;
     float m = -INFINITY, l = 0.f, acc[kSaMaxPerLane];
 #pragma unroll
     for (int i = 0; i < kSaMaxPerLane; ++i) acc[i] = 0.f;
@@ -92,10 +78,10 @@ __global__ void __launch_bounds__(kSaWarps * 32) k_sink_attn(SinkAttnP p) {
         j_hi = min(pos + 1, j_lo + per);
     }
     const float* bias = p.dist_bias ? p.dist_bias + (size_t)h * p.n_dist : nullptr;
-    for (int j = j_lo + warp; j < j_hi; j += kSaWarps) {
+    for (int j = j_lo + wm; j < j_hi; j += WPM) {
         const T* kr = kc + (size_t)j * kst;
         float s = 0.f;
-        for (int c = lane; c < p.d; c += 32) s = fmaf(sq[c], to_f32<T>(kr[c]), s);
+        for (int c = lane; c < p.d; c += 32) s = fmaf(sqm[c], to_f32<T>(kr[c]), s);
         s = warp_sum(s);
         if (bias) s += bias[min(pos - j, p.n_dist - 1)];
         const float mn = fmaxf(m, s), corr = expf(m - mn), w = expf(s - mn);
@@ -116,17 +102,48 @@ __global__ void __launch_bounds__(kSaWarps * 32) k_sink_attn(SinkAttnP p) {
     }
     __syncthreads();
     if (p.splits > 1) {   // partial result of this range, without the sink
-        float M = -INFINITY;
-        for (int w = 0; w < kSaWarps; ++w) M = fmaxf(M, sm_m[w]);
-        float L = 0.f;
-        for (int w = 0; w < kSaWarps; ++w) L = fmaf(sm_l[w], sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M), L);
-        float* part = p.ws + (((size_t)t * p.H + h) * p.splits + blockIdx.z) * (2 + p.vd);
-        if (threadIdx.x == 0) part[0] = M, part[1] = L;
-        for (int c = threadIdx.x; c < p.vd; c += blockDim.x) {
-            float o = 0.f;
-            for (int w = 0; w < kSaWarps; ++w)
-                o = fmaf(sm_acc[(size_t)w * p.vd + c], sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M), o);
-            part[2 + c] = o;
+        for (int mp = 0; mp < MAPS; ++mp) {
+            const int w0 = mp * WPM, w1 = w0 + WPM;
+            float M = -INFINITY;
+            for (int w = w0; w < w1; ++w) M = fmaxf(M, sm_m[w]);
+            float L = 0.f;
+            for (int w = w0; w < w1; ++w) L = fmaf(sm_l[w], sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M), L);
+            float* part = p.ws + ((((size_t)t * p.H + h) * MAPS + mp) * p.splits + blockIdx.z) * (2 + p.vd);
+            if (threadIdx.x == 0) part[0] = M, part[1] = L;
+            for (int c = threadIdx.x; c < p.vd; c += blockDim.x) {
+                float o = 0.f;
+                for (int w = w0; w < w1; ++w)
+                    o = fmaf(sm_acc[(size_t)w * p.vd + c], sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M), o);
+                part[2 + c] = o;
+            }
+        }
+        return;
+    }
+    if constexpr (MAPS == 2) {   // vd <= 256: one channel per thread
+        __shared__ float red[kSaWarps];
+        float a[2];
+        const int c = threadIdx.x;
+        for (int mp = 0; mp < 2; ++mp) {
+            const int w0 = mp * WPM, w1 = w0 + WPM;
+            float M = -INFINITY, L = 0.f, o = 0.f;
+            for (int w = w0; w < w1; ++w) M = fmaxf(M, sm_m[w]);
+            for (int w = w0; w < w1; ++w) {
+                const float e = sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M);
+                L = fmaf(sm_l[w], e, L);
+                if (c < p.vd) o = fmaf(sm_acc[(size_t)w * p.vd + c], e, o);
+            }
+            a[mp] = o / L;
+        }
+        const float o = c < p.vd ? a[0] - p.lambda * a[1] : 0.f;
+        const float ws = warp_sum(o * o);
+        if (lane == 0) red[warp] = ws;
+        __syncthreads();
+        float ss = 0.f;
+        for (int w = 0; w < kSaWarps; ++w) ss += red[w];
+        if (c < p.vd) {
+            float v = o * (p.out_mul / sqrtf(ss / (float)p.vd + p.out_eps));
+            if (p.gate_full) v *= sa_sigmoid(p.gate_full[(size_t)t * p.ldg + (size_t)h * p.vd + c]);
+            static_cast<T*>(p.out)[((size_t)t * p.H + h) * p.vd + c] = from_f32<T>(v);
         }
         return;
     }
@@ -168,22 +185,6 @@ struct SinkAttnMmaP {
 
 constexpr int kTq = 64, kTk = 64;
 
-__device__ __forceinline__ void sa_cp_async16(void* smem_dst, const void* gsrc) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem_dst)), "l"(gsrc) : "memory");
-}
-__device__ __forceinline__ void sa_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void sa_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void sa_ldmatrix_x4(uint32_t (&r)[4], const void* smem_row) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(smem_u32(smem_row)));
-}
-__device__ __forceinline__ void sa_ldmatrix_x4_trans(uint32_t (&r)[4], const void* smem_row) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(smem_u32(smem_row)));
-}
 template <typename T>
 __device__ __forceinline__ void sa_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1);
 template <>
@@ -194,30 +195,28 @@ template <>
 __device__ __forceinline__ void sa_mma<__nv_bfloat16>(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     mma_16816_bf16(d, a, b0, b1, d);
 }
-template <typename T>
-__device__ __forceinline__ uint32_t sa_pack(float x, float y) {
-    T a = from_f32<T>(x), b = from_f32<T>(y);
-    return (uint32_t) * reinterpret_cast<uint16_t*>(&a) | ((uint32_t) * reinterpret_cast<uint16_t*>(&b) << 16);
-}
-
 // grid (ceil(longest run / tokens per tile), G, runs * splits); 4 warps.  NV: 8-column value tiles per warp.
 // DEC = false: a tile of 64 rows, 16 per warp, every warp over all 64 keys of a key tile.
 // DEC = true (the rows of a tile fit 16: decode steps): every warp holds the same 16 rows and takes 16 of the 64 keys
 // of a key tile with a softmax state of its own; the four states are merged through shared memory at the end.
-template <typename T, int NV, bool DEC>
+// MAPS = 2: the first half of the warps works on the first map, the second on the second; a key tile holds both maps' keys.
+// DEC = false: 32 rows per map.  DEC = true: 16 rows per map, a warp takes 32 of the 64 keys.
+template <typename T, int NV, bool DEC, int MAPS>
 __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     extern __shared__ __align__(16) unsigned char sa_raw[];
     const SinkAttnP& p = pp.a;
-    constexpr int QR = DEC ? 16 : kTq;      // rows of the query tile
-    constexpr int NS = DEC ? 2 : 8;         // 8-key score tiles per warp and key tile
-    const int DP = p.d + 8, VP = NV * 8 + 8;
+    constexpr int QM = DEC ? 16 : kTq / MAPS;   // rows of the query tile per map
+    constexpr int QR = QM * MAPS;
+    constexpr int WPM = 4 / MAPS;               // warps per map
+    constexpr int NS = DEC ? 8 / WPM : 8;       // 8-key score tiles per warp and key tile
+    const int DP = p.d + 8, KP = MAPS * p.d + 8, VP = NV * 8 + 8;
     T* sQ = reinterpret_cast<T*>(sa_raw);   // [QR][DP]
-    T* sK = sQ + QR * DP;                   // [2][kTk][DP]
-    T* sV = sK + 2 * kTk * DP;              // [2][kTk][VP]
+    T* sK = sQ + QR * DP;                   // [2][kTk][KP]
+    T* sV = sK + 2 * kTk * KP;              // [2][kTk][VP]
     pdl_trigger();
     pdl_wait();
     const int run = blockIdx.z / p.splits, split = blockIdx.z % p.splits, g = blockIdx.y;
-    const int R = p.H / p.G, nq = QR / R;
+    const int R = p.H / p.G, nq = QM / R;
     const int len = pp.run_len[run], t0 = blockIdx.x * nq;
     if (t0 >= len) return;
     const int ntok = min(nq, len - t0), row0 = pp.run_row0[run] + t0;
@@ -231,18 +230,18 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
         k_hi = min(n_keys, k_lo + per);
     }
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
-    const int d8 = p.d >> 3, v8 = p.vd >> 3;
-    const T* kc = static_cast<const T*>(p.k_addrs[sl]) + (size_t)g * p.d;
+    const int d8 = p.d >> 3, k8 = MAPS * d8, v8 = p.vd >> 3;
+    const T* kc = static_cast<const T*>(p.k_addrs[sl]) + (size_t)g * MAPS * p.d;
     const T* vc = static_cast<const T*>(p.v_addrs[sl]) + (size_t)g * p.vd;
-    const size_t kst = (size_t)p.G * p.d, vst = (size_t)p.G * p.vd;
+    const size_t kst = (size_t)p.G * MAPS * p.d, vst = (size_t)p.G * p.vd;
 
     auto load_kv = [&](int buf, int k0) {
-        T* dk = sK + (size_t)buf * kTk * DP;
+        T* dk = sK + (size_t)buf * kTk * KP;
         T* dv = sV + (size_t)buf * kTk * VP;
-        for (int i = tid; i < kTk * d8; i += 128) {
-            const int r = i / d8, c = i - r * d8, kj = k0 + r;
-            if (kj < k_hi) sa_cp_async16(dk + (size_t)r * DP + c * 8, kc + (size_t)kj * kst + c * 8);
-            else *reinterpret_cast<uint4*>(dk + (size_t)r * DP + c * 8) = make_uint4(0, 0, 0, 0);
+        for (int i = tid; i < kTk * k8; i += 128) {
+            const int r = i / k8, c = i - r * k8, kj = k0 + r;
+            if (kj < k_hi) sa_cp_async16(dk + (size_t)r * KP + c * 8, kc + (size_t)kj * kst + c * 8);
+            else *reinterpret_cast<uint4*>(dk + (size_t)r * KP + c * 8) = make_uint4(0, 0, 0, 0);
         }
         for (int i = tid; i < kTk * (NV + 0); i += 128) {
             const int r = i / NV, c = i - r * NV, kj = k0 + r;
@@ -250,8 +249,10 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
             else *reinterpret_cast<uint4*>(dv + (size_t)r * VP + c * 8) = make_uint4(0, 0, 0, 0);
         }
     };
-    // rows of this thread: wrow + gq and + 8; row -> (token, head in the group).  kb: the warp's first key in a key tile
-    const int wrow = DEC ? 0 : warp * 16, kb = DEC ? warp * 16 : 0;
+    // rows of this thread: wrow + gq and + 8 among the map's rows; row -> (token, head in the group).  kb: the warp's first
+    // key in a key tile
+    const int map = warp / WPM, wm = warp - map * WPM;
+    const int wrow = DEC ? 0 : wm * 16, kb = DEC ? wm * (kTk / WPM) : 0;
     int tok_of[2], pos_of[2], head_of[2], first_of[2];
     bool row_ok[2];
     const float* bias_of[2];
@@ -280,10 +281,10 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     if (k_lo < k_hi) {
         // the query tile
         for (int i = tid; i < QR * d8; i += 128) {
-            const int r = i / d8, c = i - r * d8, tk = r / R;
+            const int r = i / d8, c = i - r * d8, mp = r / QM, rm = r - mp * QM, tk = rm / R;
             uint4 v = make_uint4(0, 0, 0, 0);
             if (tk < ntok)
-                v = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.q) + ((size_t)(row0 + tk) * p.H + g * R + (r - tk * R)) * p.d + c * 8);
+                v = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.q) + (((size_t)(row0 + tk) * p.H + g * R + (rm - tk * R)) * MAPS + mp) * p.d + c * 8);
             *reinterpret_cast<uint4*>(sQ + (size_t)r * DP + c * 8) = v;
         }
         load_kv(0, k_lo);
@@ -294,7 +295,7 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
             __syncthreads();   // tile k0 (and the query tile) is in shared memory; every warp is done with the other buffer
             if (k0 + kTk < k_hi) load_kv(buf ^ 1, k0 + kTk);
             sa_cp_commit();
-            const T* tK = sK + (size_t)buf * kTk * DP;
+            const T* tK = sK + (size_t)buf * kTk * KP + map * p.d;
             const T* tV = sV + (size_t)buf * kTk * VP;
             float S[NS][4];
 #pragma unroll
@@ -303,11 +304,11 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
                 for (int c = 0; c < 4; ++c) S[j][c] = 0.f;
             for (int kk = 0; kk < p.d; kk += 16) {
                 uint32_t a[4];
-                sa_ldmatrix_x4(a, sQ + (size_t)(wrow + (lane & 15)) * DP + kk + (lane >> 4) * 8);
+                sa_ldmatrix_x4(a, sQ + (size_t)(map * QM + wrow + (lane & 15)) * DP + kk + (lane >> 4) * 8);
 #pragma unroll
                 for (int jj = 0; jj < NS / 2; ++jj) {
                     uint32_t b[4];
-                    sa_ldmatrix_x4(b, tK + (size_t)(kb + jj * 16 + (lane & 7) + (lane >> 4) * 8) * DP + kk + ((lane >> 3) & 1) * 8);
+                    sa_ldmatrix_x4(b, tK + (size_t)(kb + jj * 16 + (lane & 7) + (lane >> 4) * 8) * KP + kk + ((lane >> 3) & 1) * 8);
                     sa_mma<T>(S[2 * jj], a, b[0], b[1]);
                     sa_mma<T>(S[2 * jj + 1], a, b[2], b[3]);
                 }
@@ -401,6 +402,53 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
         const int r = tid >> 3, tk = r / R;   // 8 threads per row
         if (tk >= ntok) return;
         const int t = row0 + tk, h = g * R + (r - tk * R);
+        if constexpr (MAPS == 2) {
+            float wg[4], ML[2], LL[2];
+#pragma unroll
+            for (int mp = 0; mp < 2; ++mp) {
+                float M = -1e30f, L = 0.f;
+#pragma unroll
+                for (int w = mp * 2; w < mp * 2 + 2; ++w) M = fmaxf(M, mm[w * 16 + r]);
+#pragma unroll
+                for (int w = mp * 2; w < mp * 2 + 2; ++w) {
+                    wg[w] = ml[w * 16 + r] > 0.f ? expf(mm[w * 16 + r] - M) : 0.f;
+                    L = fmaf(ml[w * 16 + r], wg[w], L);
+                }
+                ML[mp] = M, LL[mp] = L;
+            }
+            auto val = [&](int w, int c) { return mo[((size_t)w * 16 + r) * (NV * 8) + c] * wg[w]; };
+            if (p.splits > 1) {
+#pragma unroll
+                for (int mp = 0; mp < 2; ++mp) {
+                    float* part = p.ws + ((((size_t)t * p.H + h) * 2 + mp) * p.splits + split) * (2 + p.vd);
+                    if ((tid & 7) == 0) part[0] = LL[mp] > 0.f ? ML[mp] : -INFINITY, part[1] = LL[mp];
+                    for (int c = tid & 7; c < p.vd; c += 8) part[2 + c] = val(2 * mp, c) + val(2 * mp + 1, c);
+                }
+                return;
+            }
+            float keep[NV], ss = 0.f;
+            const float i0 = 1.0f / LL[0], i1 = p.lambda / LL[1];
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = (tid & 7) + 8 * i;
+                keep[i] = c < p.vd ? (val(0, c) + val(1, c)) * i0 - (val(2, c) + val(3, c)) * i1 : 0.f;
+                ss = fmaf(keep[i], keep[i], ss);
+            }
+            const uint32_t act = 0xffu << (lane & 24);   // the 8 threads of this row
+#pragma unroll
+            for (int o = 1; o < 8; o <<= 1) ss += __shfl_xor_sync(act, ss, o);
+            const float mul = p.out_mul / sqrtf(ss / (float)p.vd + p.out_eps);
+            T* out = static_cast<T*>(p.out) + ((size_t)t * p.H + h) * p.vd;
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = (tid & 7) + 8 * i;
+                if (c >= p.vd) continue;
+                float v = keep[i] * mul;
+                if (p.gate_full) v *= sa_sigmoid(p.gate_full[(size_t)t * p.ldg + (size_t)h * p.vd + c]);
+                out[c] = from_f32<T>(v);
+            }
+            return;
+        }
         const float sink = p.sink ? p.sink[h] : 0.f;
         const bool with_sink = p.splits == 1 && !p.no_sink;
         float M = with_sink ? sink : -1e30f;
@@ -443,6 +491,48 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
             }
         }
     } else {
+    if constexpr (MAPS == 2) {
+        if (p.splits == 1) {
+            // both maps' normalised rows through shared memory, then one warp per (token, head)
+            __syncthreads();
+            float* so = reinterpret_cast<float*>(sa_raw);   // [kTq][vd + 1]
+            const int SP = p.vd + 1;
+#pragma unroll
+            for (int hh = 0; hh < 2; ++hh) {
+                if (!row_ok[hh]) continue;
+                const float inv = (map ? p.lambda : 1.0f) / l_run[hh];
+                float* sr = so + (size_t)(map * QM + wrow + gq + hh * 8) * SP;
+#pragma unroll
+                for (int j = 0; j < NV; ++j) {
+                    const int c = 8 * j + 2 * tq;
+                    if (c < p.vd) sr[c] = O[j][hh * 2] * inv, sr[c + 1] = O[j][hh * 2 + 1] * inv;
+                }
+            }
+            __syncthreads();
+            for (int r = warp; r < ntok * R; r += 4) {
+                const int tk = r / R, t = row0 + tk, h = g * R + (r - tk * R);
+                const float *a1 = so + (size_t)r * SP, *a2 = so + (size_t)(QM + r) * SP;
+                float keep[NV / 4], ss = 0.f;
+#pragma unroll
+                for (int i = 0; i < NV / 4; ++i) {
+                    const int c = lane + 32 * i;
+                    keep[i] = c < p.vd ? a1[c] - a2[c] : 0.f;
+                    ss = fmaf(keep[i], keep[i], ss);
+                }
+                const float mul = p.out_mul / sqrtf(warp_sum(ss) / (float)p.vd + p.out_eps);
+                T* out = static_cast<T*>(p.out) + ((size_t)t * p.H + h) * p.vd;
+#pragma unroll
+                for (int i = 0; i < NV / 4; ++i) {
+                    const int c = lane + 32 * i;
+                    if (c >= p.vd) continue;
+                    float v = keep[i] * mul;
+                    if (p.gate_full) v *= sa_sigmoid(p.gate_full[(size_t)t * p.ldg + (size_t)h * p.vd + c]);
+                    out[c] = from_f32<T>(v);
+                }
+            }
+            return;
+        }
+    }
     if (p.out_table && p.splits == 1) {
         // the tile's normalised rows go through shared memory (the key tiles are no longer needed): the two channels of a
         // pair sit in different threads
@@ -480,7 +570,7 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
         if (!row_ok[hh]) continue;
         const int t = row0 + tok_of[hh], h = head_of[hh];
         if (p.splits > 1) {
-            float* part = p.ws + (((size_t)t * p.H + h) * p.splits + split) * (2 + p.vd);
+            float* part = p.ws + ((((size_t)t * p.H + h) * MAPS + map) * p.splits + split) * (2 + p.vd);
             const bool empty = l_run[hh] <= 0.f;
             if (tq == 0) part[0] = empty ? -INFINITY : m_run[hh], part[1] = empty ? 0.f : l_run[hh];
 #pragma unroll
@@ -506,32 +596,32 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     }
 }
 
-template <typename T, int NV, bool DEC>
+template <typename T, int NV, bool DEC, int MAPS>
 static cudaError_t launch_sink_mma(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
     const SinkAttnP& p = pp.a;
-    const int qr = DEC ? 16 : kTq, nq = qr / (p.H / p.G);
-    size_t smem = ((size_t)qr * (p.d + 8) + 2 * (size_t)kTk * (p.d + 8) + 2 * (size_t)kTk * (NV * 8 + 8)) * sizeof(T);
+    const int qm = DEC ? 16 : kTq / MAPS, nq = qm / (p.H / p.G);
+    size_t smem = ((size_t)qm * MAPS * (p.d + 8) + 2 * (size_t)kTk * (MAPS * p.d + 8) + 2 * (size_t)kTk * (NV * 8 + 8)) * sizeof(T);
     if (DEC && smem < (size_t)(128 + 64 * NV * 8) * sizeof(float)) smem = (size_t)(128 + 64 * NV * 8) * sizeof(float);
-    if (!DEC && p.out_table && smem < (size_t)kTq * (p.vd + 1) * sizeof(float)) smem = (size_t)kTq * (p.vd + 1) * sizeof(float);
+    if (!DEC && (p.out_table || MAPS == 2) && smem < (size_t)kTq * (p.vd + 1) * sizeof(float)) smem = (size_t)kTq * (p.vd + 1) * sizeof(float);
     static size_t set_for = 0;
     if (smem > 48 * 1024 && smem > set_for) {
-        const cudaError_t e = cudaFuncSetAttribute(k_sink_attn_mma<T, NV, DEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(k_sink_attn_mma<T, NV, DEC, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
         set_for = smem;
     }
-    return launch(k_sink_attn_mma<T, NV, DEC>, dim3(cdiv(max_run_len, nq), p.G, runs * p.splits), dim3(128), smem, st, pdl, pp);
+    return launch(k_sink_attn_mma<T, NV, DEC, MAPS>, dim3(cdiv(max_run_len, nq), p.G, runs * p.splits), dim3(128), smem, st, pdl, pp);
 }
-template <typename T, int NV>
+template <typename T, int NV, int MAPS>
 static cudaError_t launch_sink_mma_d(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
     // the rows of the longest run fit one 16-row tile: the decode form
-    if (max_run_len * (pp.a.H / pp.a.G) <= 16) return launch_sink_mma<T, NV, true>(pp, runs, max_run_len, pdl, st);
-    return launch_sink_mma<T, NV, false>(pp, runs, max_run_len, pdl, st);
+    if (max_run_len * (pp.a.H / pp.a.G) <= 16) return launch_sink_mma<T, NV, true, MAPS>(pp, runs, max_run_len, pdl, st);
+    return launch_sink_mma<T, NV, false, MAPS>(pp, runs, max_run_len, pdl, st);
 }
-template <typename T>
+template <typename T, int MAPS>
 static cudaError_t launch_sink_mma_t(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
-    if (pp.a.vd <= 32) return launch_sink_mma_d<T, 4>(pp, runs, max_run_len, pdl, st);
-    if (pp.a.vd <= 64) return launch_sink_mma_d<T, 8>(pp, runs, max_run_len, pdl, st);
-    return launch_sink_mma_d<T, 16>(pp, runs, max_run_len, pdl, st);
+    if (pp.a.vd <= 32) return launch_sink_mma_d<T, 4, MAPS>(pp, runs, max_run_len, pdl, st);
+    if (pp.a.vd <= 64) return launch_sink_mma_d<T, 8, MAPS>(pp, runs, max_run_len, pdl, st);
+    return launch_sink_mma_d<T, 16, MAPS>(pp, runs, max_run_len, pdl, st);
 }
 
 // merge of the splits (at most 32) with the sink term and the gate; one warp per (token, head), grid (ceil(H / 4), T).
@@ -585,6 +675,83 @@ __global__ void __launch_bounds__(128) k_sink_attn_merge(SinkAttnP p) {
         for (int s = 0; s < 32; ++s) o = fmaf(v[s], wv[s], o);   // splits in order; absent ones add 0 * 0
         out[c] = from_f32<T>(o / L * gate);
     }
+}
+
+// the same for two maps per head: both maps' merged results meet, then the norm over the head and the gate
+template <typename T>
+__global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.y, h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (h >= p.H) return;
+    const int stride = 2 + p.vd;
+    float keep[kSaMaxPerLane], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kSaMaxPerLane; ++i) keep[i] = 0.f;
+    for (int mp = 0; mp < 2; ++mp) {
+        const float* part = p.ws + (((size_t)t * p.H + h) * 2 + mp) * p.splits * stride;
+        const float ms = lane < p.splits ? part[(size_t)lane * stride] : -INFINITY;
+        const float ls = lane < p.splits ? part[(size_t)lane * stride + 1] : 0.f;
+        const float M = warp_max(ms);
+        const float wgt = ms == -INFINITY ? 0.f : expf(ms - M);
+        float L = 0.f, wv[32];
+#pragma unroll
+        for (int s = 0; s < 32; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
+        for (int s = 0; s < p.splits; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, wgt, s), L);
+        const float f = (mp ? -p.lambda : 1.0f) / L;
+#pragma unroll
+        for (int i = 0; i < kSaMaxPerLane; ++i) {
+            const int c = lane + 32 * i;
+            if (c >= p.vd) continue;
+            float v[32];
+#pragma unroll
+            for (int s = 0; s < 32; ++s) v[s] = s < p.splits ? part[(size_t)s * stride + 2 + c] : 0.f;   // all loads in flight
+            float o = 0.f;
+#pragma unroll
+            for (int s = 0; s < 32; ++s) o = fmaf(v[s], wv[s], o);
+            keep[i] = fmaf(o, f, keep[i]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < kSaMaxPerLane; ++i) ss = fmaf(keep[i], keep[i], ss);
+    const float mul = p.out_mul / sqrtf(warp_sum(ss) / (float)p.vd + p.out_eps);
+    T* out = static_cast<T*>(p.out) + ((size_t)t * p.H + h) * p.vd;
+#pragma unroll
+    for (int i = 0; i < kSaMaxPerLane; ++i) {
+        const int c = lane + 32 * i;
+        if (c >= p.vd) continue;
+        float v = keep[i] * mul;
+        if (p.gate_full) v *= sa_sigmoid(p.gate_full[(size_t)t * p.ldg + (size_t)h * p.vd + c]);
+        out[c] = from_f32<T>(v);
+    }
+}
+
+template <typename T>
+static cudaError_t sa_merge_t(const SinkAttnP& p, int maps, int T_, bool pdl, cudaStream_t st) {
+    const dim3 mg(cdiv(p.H, 4), T_), mb(128);
+    return maps == 2 ? launch(k_two_map_merge<T>, mg, mb, 0, st, pdl, p) : launch(k_sink_attn_merge<T>, mg, mb, 0, st, pdl, p);
+}
+int sink_attn_merge(const SinkAttnP& p, int maps, int T, int dtype, bool pdl, cudaStream_t st) {
+    cudaError_t e;
+    if (dtype == ZL_F32) e = sa_merge_t<float>(p, maps, T, pdl, st);
+    else if (dtype == ZL_BF16) e = sa_merge_t<__nv_bfloat16>(p, maps, T, pdl, st);
+    else e = sa_merge_t<__half>(p, maps, T, pdl, st);
+    ZL_CHECK_CUDA(e);
+    return ZL_OK;
+}
+
+template <typename T, int MAPS>
+static cudaError_t launch_sink_general(const SinkAttnP& p, int T_, bool pdl, cudaStream_t st) {
+    const size_t smem = ((size_t)MAPS * p.d + 2 * kSaWarps + (size_t)kSaWarps * p.vd) * sizeof(float);
+    return launch(k_sink_attn<T, MAPS>, dim3(p.H, T_, p.splits), dim3(kSaWarps * 32), smem, st, pdl, p);
+}
+
+static bool sink_mma_eligible(const SinkAttnP& p, const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len,
+                              int maps, int dtype) {
+    static const bool no_mma = getenv("ZL_SINK_ATTN_NO_MMA") != nullptr;
+    const int R = p.H / p.G;
+    return !no_mma && run_row0 && run_len && runs > 0 && max_run_len > 0 && dtype != ZL_F32 && p.d % 16 == 0 && p.vd % 8 == 0 &&
+           p.vd <= 128 && maps * p.d <= 256 && R <= 16 && 16 % R == 0;
 }
 
 }  // namespace zl
@@ -666,27 +833,59 @@ extern "C" int zl_sink_attention_ex(const void* q, void* const* k_addrs, void* c
     p.no_sink = no_sink != 0;
     p.out_table = out_table;
     p.out_layout = out_layout;
-    const dim3 grid(heads, T, splits), block(kSaWarps * 32);
-    const size_t smem = ((size_t)dim + 2 * kSaWarps + (size_t)kSaWarps * vdim) * sizeof(float);
     cudaError_t e;
-    static const bool no_mma = getenv("ZL_SINK_ATTN_NO_MMA") != nullptr;
-    const bool mma = !no_mma && run_row0 && run_len && runs > 0 && max_run_len > 0 && dtype != ZL_F32 && dim % 16 == 0 &&
-                     vdim % 8 == 0 && vdim <= 128 && dim <= 256 && heads / kv_heads <= 16 && 16 % (heads / kv_heads) == 0;
-    if (mma) {
+    if (sink_mma_eligible(p, run_row0, run_len, runs, max_run_len, 1, dtype)) {
         ZL_CHECK_ARG((long long)runs * splits <= 65535 && kv_heads <= 65535);
         SinkAttnMmaP pp{p, run_row0, run_len};
-        e = dtype == ZL_BF16 ? launch_sink_mma_t<__nv_bfloat16>(pp, runs, max_run_len, pdl != 0, stream)
-                             : launch_sink_mma_t<__half>(pp, runs, max_run_len, pdl != 0, stream);
-    } else if (dtype == ZL_F32) e = launch(k_sink_attn<float>, grid, block, smem, stream, pdl != 0, p);
-    else if (dtype == ZL_BF16) e = launch(k_sink_attn<__nv_bfloat16>, grid, block, smem, stream, pdl != 0, p);
-    else e = launch(k_sink_attn<__half>, grid, block, smem, stream, pdl != 0, p);
+        e = dtype == ZL_BF16 ? launch_sink_mma_t<__nv_bfloat16, 1>(pp, runs, max_run_len, pdl != 0, stream)
+                             : launch_sink_mma_t<__half, 1>(pp, runs, max_run_len, pdl != 0, stream);
+    } else if (dtype == ZL_F32) e = launch_sink_general<float, 1>(p, T, pdl != 0, stream);
+    else if (dtype == ZL_BF16) e = launch_sink_general<__nv_bfloat16, 1>(p, T, pdl != 0, stream);
+    else e = launch_sink_general<__half, 1>(p, T, pdl != 0, stream);
     ZL_CHECK_CUDA(e);
-    if (splits > 1) {
-        const dim3 mg(cdiv(heads, 4), T), mb(128);
-        if (dtype == ZL_F32) e = launch(k_sink_attn_merge<float>, mg, mb, 0, stream, pdl != 0, p);
-        else if (dtype == ZL_BF16) e = launch(k_sink_attn_merge<__nv_bfloat16>, mg, mb, 0, stream, pdl != 0, p);
-        else e = launch(k_sink_attn_merge<__half>, mg, mb, 0, stream, pdl != 0, p);
-        ZL_CHECK_CUDA(e);
+    return splits > 1 ? sink_attn_merge(p, 1, T, dtype, pdl != 0, stream) : ZL_OK;
+}
+
+extern "C" int zl_window_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot,
+                                   const int32_t* pos, float scale, int window, int maps, float lambda, float out_eps,
+                                   float out_mul, const float* gate, long long ldg, void* out, int T, int heads, int kv_heads,
+                                   int dim, int vdim, int splits, void* workspace, size_t workspace_bytes,
+                                   const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
+                                   zl_stream_t stream) {
+    ZL_CHECK_ARG(q && k_addrs && v_addrs && slot && pos && out && T > 0 && T <= 65535 && heads > 0 && kv_heads > 0);
+    ZL_CHECK_ARG(heads % kv_heads == 0 && dim > 0 && vdim > 0 && window >= 0 && (maps == 1 || maps == 2) && out_eps >= 0.f);
+    ZL_CHECK_ARG(maps == 2 || !gate);
+    ZL_CHECK_SUPPORTED(vdim <= 32 * kSaMaxPerLane && dim <= 2048);
+    ZL_CHECK_ARG(dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32);
+    ZL_CHECK_ARG(splits >= 1 && splits <= 32);
+    ZL_CHECK_ARG(splits == 1 || (workspace && workspace_bytes >= zl_sink_attention_workspace_bytes(T, heads * maps, vdim, splits)));
+    SinkAttnP p{q, k_addrs, v_addrs, slot, pos, nullptr, nullptr, ldg, out, heads, kv_heads, dim, vdim, scale, splits,
+                static_cast<float*>(workspace)};
+    p.no_sink = 1;
+    p.window = window;
+    p.lambda = lambda;
+    p.out_eps = out_eps;
+    p.out_mul = out_mul;
+    p.gate_full = gate;
+    cudaError_t e;
+    if (sink_mma_eligible(p, run_row0, run_len, runs, max_run_len, maps, dtype)) {
+        ZL_CHECK_ARG((long long)runs * splits <= 65535 && kv_heads <= 65535);
+        SinkAttnMmaP pp{p, run_row0, run_len};
+        if (maps == 2)
+            e = dtype == ZL_BF16 ? launch_sink_mma_t<__nv_bfloat16, 2>(pp, runs, max_run_len, pdl != 0, stream)
+                                 : launch_sink_mma_t<__half, 2>(pp, runs, max_run_len, pdl != 0, stream);
+        else
+            e = dtype == ZL_BF16 ? launch_sink_mma_t<__nv_bfloat16, 1>(pp, runs, max_run_len, pdl != 0, stream)
+                                 : launch_sink_mma_t<__half, 1>(pp, runs, max_run_len, pdl != 0, stream);
+    } else if (maps == 2) {
+        if (dtype == ZL_F32) e = launch_sink_general<float, 2>(p, T, pdl != 0, stream);
+        else if (dtype == ZL_BF16) e = launch_sink_general<__nv_bfloat16, 2>(p, T, pdl != 0, stream);
+        else e = launch_sink_general<__half, 2>(p, T, pdl != 0, stream);
+    } else {
+        if (dtype == ZL_F32) e = launch_sink_general<float, 1>(p, T, pdl != 0, stream);
+        else if (dtype == ZL_BF16) e = launch_sink_general<__nv_bfloat16, 1>(p, T, pdl != 0, stream);
+        else e = launch_sink_general<__half, 1>(p, T, pdl != 0, stream);
     }
-    return ZL_OK;
+    ZL_CHECK_CUDA(e);
+    return splits > 1 ? sink_attn_merge(p, maps, T, dtype, pdl != 0, stream) : ZL_OK;
 }

@@ -104,6 +104,16 @@ def _build_dizizen(config, dtype, max_batch, max_seq, max_step_tokens, **kw):
 register("Dizizen", _build_dizizen, ("bfloat16", "float32"))
 
 
+# ---- Dekalorn --------------------------------------------------------------------------------------------------------
+def _build_dekalorn(config, dtype, max_batch, max_seq, max_step_tokens, **kw):
+    from .dekalorn import DekalornDecoder
+    return DekalornDecoder.from_config_dict(config, dtype=dtype, max_batch=max_batch, max_seq=max_seq,
+                                            max_step_tokens=max_step_tokens, **kw)
+
+
+register("Dekalorn", _build_dekalorn, ("bfloat16", "float32"))
+
+
 # ---- Llama (HF folder) -----------------------------------------------------------------------------------------------
 _HF_LLAMA_NAMES = [
     (r"^model\.embed_tokens\.weight$", "token_embedding.weight"),
