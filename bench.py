@@ -809,6 +809,135 @@ def run_compare_dizizen(args):
                       "timing": "CUDA events on the model's stream; weights per pass larger than L2"}))
 
 
+# ----------------------------------------------------------------------------------------------------------------------
+# --compare-dekalorn: prefill and decode throughput of the Dekalorn family beside Kodupel (the closest existing model:
+# attention over slot caches, silu-like gated experts of three matrices, an fp32 residual stream, the same GEMM / routing
+# kernels) at equal width, depth, heads and feed-forward parameters per token, random weights; --compare-models may add
+# "dekipel" (the other family with latent attention).  Does not touch the default workload.
+# ----------------------------------------------------------------------------------------------------------------------
+DEKALORN_RANK, DEKALORN_ROT, DEKALORN_WINDOW = 512, 64, 1024
+
+
+def _dekalorn_config(sz):
+    """Layers: latent / dense, differential / experts, mixed heads / experts, latent / experts, as one pass of a loop."""
+    H, d = sz["heads"], sz["dim"]
+    moe = {"kind": "moe", "expert": {"ff": sz["ff_e"]},
+           "router": {"experts": sz["experts"], "top": sz["top"], "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    latent = {"type": "latent_attention",
+              "mixer": dict(heads=H, dim=d, rot_dim=DEKALORN_ROT, vdim=d, kv_rank=DEKALORN_RANK, scale=(d + DEKALORN_ROT) ** -0.5,
+                            rot={"base": 1e4, "dims": DEKALORN_ROT})}
+    diff = {"type": "attention",
+            "mixer": dict(heads=H, kv_heads=8, dim=d // 2, vdim=d, scale=(d // 2) ** -0.5, diff=0.4, mask={"size": DEKALORN_WINDOW})}
+    mixed = {"type": "attention_2",
+             "mixer": dict(heads=H, kv_heads=8, dim=d, vdim=d, scale=d ** -0.5, mask={"size": DEKALORN_WINDOW},
+                           rot={"base": 5e5, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})}
+    kinds = [(latent, {"kind": "dense", "ff": sz["ff"]}), (diff, moe), (mixed, moe), (latent, moe)]
+    layers = [dict(kinds[i % 4][0], mlp=kinds[i % 4][1]) for i in range(sz["layers"])]
+    return {"architecture": "Dekalorn", "vocab": sz["vocab"], "width": sz["width"], "layers": layers, "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": len(layers), "times": 1}}
+
+
+def _dekalorn_params(sz, rows, ctx):
+    """(Linear parameters one token uses, parameters a step of `rows` tokens reads, cache bytes a token at `ctx` reads)."""
+    D, H, d, E, top, fe = sz["width"], sz["heads"], sz["dim"], sz["experts"], sz["top"], sz["ff_e"]
+    R, r, win = DEKALORN_RANK, DEKALORN_ROT, min(ctx, DEKALORN_WINDOW)
+    touched = E * (1.0 - (1.0 - top / E) ** rows)
+    mix = {0: D * (H * (d + r) + R + r + H) + 2 * H * d * R + H * d * D, 1: D * (H * d + 8 * d + 8 * d + H * d) + H * d * D,
+           2: D * (H * d + 2 * 8 * d) + H * d * D}
+    rows_of = {0: ctx * (R + r) * 2, 1: win * 8 * 2 * d * 2, 2: win * 8 * 2 * d * 2}
+    active = read = 2 * D * D + sz["vocab"] * D
+    cache = 0
+    for i in range(sz["layers"]):
+        k = (0, 1, 2, 0)[i % 4]
+        active += mix[k] + (3 * D * sz["ff"] if i % 4 == 0 else E * D + top * 3 * D * fe)
+        read += mix[k] + (3 * D * sz["ff"] if i % 4 == 0 else E * D + touched * 3 * D * fe)
+        cache += rows_of[k]
+    return active, read, cache
+
+
+def run_compare_dekalorn(args):
+    import numpy as np
+    import torch
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: the hot path has no CPU fallback")
+    torch.cuda.set_device(0)
+    from zhilight_b200 import build
+    build.build()
+    from zhilight_b200.dekalorn import DekalornDecoder
+    from zhilight_b200.dekipel import DekipelDecoder
+    from zhilight_b200.kodupel import KodupelDecoder
+    hbm, how = read_peaks()
+    peaks_path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = json.load(open(peaks_path))["bf16_tflops"] if os.path.exists(peaks_path) else 1590.0
+    ctx, chunk, n_prompt = args.prompt if args.prompt > 128 else 1024, 1024, 2048
+    steps, warm = max(args.steps, 16), max(args.warmup, 3)
+    rng = np.random.default_rng(0)
+    rows = []
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.mark_region_start()
+    for name, sz in KODUPEL_SIZES.items():
+        if args.compare_sizes and name not in args.compare_sizes.split(","):
+            continue
+        for kind in [k for k in ("dekalorn", "kodupel", "dekipel") if k in args.compare_models.split(",")]:
+            max_seq = max(ctx, n_prompt) + 4 * (steps + warm) + 64
+            kw = dict(dtype="bf16", max_batch=32, max_seq=max_seq, max_step_tokens=chunk, use_pdl=not args.no_pdl,
+                      use_graph=not args.no_graph)
+            if kind == "dekalorn":
+                dec = DekalornDecoder.from_config_dict(_dekalorn_config(sz), **kw)
+                active = _dekalorn_params(sz, 1, ctx)[0]
+            elif kind == "kodupel":
+                dec = KodupelDecoder.from_config_dict(_kodupel_config(sz), **kw)
+                active = _kodupel_params(sz, 1)[0]
+            else:
+                dec = DekipelDecoder.from_config_dict(_dekipel_config(COMPARE_SIZES[name]), **kw)
+                active = _linear_params("dekipel", COMPARE_SIZES[name])
+            dec.init_synthetic(seed=1)
+            stream = torch.cuda.ExternalStream(dec.stream())
+            out = {"size": name, "model": kind}
+            toks = rng.integers(0, sz["vocab"], n_prompt).astype(np.int32)
+            for _ in range(2):
+                dec.prefill(0, toks, 0)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(stream)
+            for _ in range(3):
+                dec.prefill(0, toks, 0)
+            e1.record(stream)
+            e1.synchronize()
+            ms = e0.elapsed_time(e1) / 3
+            out["linear_params_per_token"] = int(active)
+            flops = 2.0 * (active - sz["vocab"] * sz["width"]) * n_prompt
+            out["prefill"] = {"tokens": n_prompt, "chunk": chunk, "ms": round(ms, 3), "tok_s": round(n_prompt / ms * 1e3),
+                              "linear_tflops": round(flops / ms / 1e9, 1),
+                              "of_measured_bf16_peak": round(flops / ms / 1e9 / tflops, 4)}
+            for b in range(32):
+                dec.prefill(b, toks[:ctx], 0)
+            for B in (1, 32):
+                dec.set_state(rng.integers(0, sz["vocab"], B).astype(np.int32), np.full(B, ctx, dtype=np.int32))
+                ms, _ = measure_decode(dec, B, steps, warm, stream, torch.cuda.synchronize)
+                mid = ctx + warm + steps // 2
+                if kind == "dekalorn":
+                    _, read, cache = _dekalorn_params(sz, B, mid)
+                    step_bytes = read * 2 + B * cache
+                elif kind == "kodupel":
+                    _, read, cache, state = _kodupel_params(sz, B)
+                    step_bytes = read * 2 + B * (mid * cache + state)
+                else:
+                    step_bytes = active * 2 + B * mid * COMPARE_SIZES[name]["kv_rank"] * 2 * ((sz["layers"] + 1) // 2)
+                out["decode_b%d" % B] = {"ctx": ctx, "ms_per_step": round(ms / steps, 4), "tok_s": round(B * steps / ms * 1e3, 1),
+                                          "step_bytes": int(step_bytes),
+                                          "of_%s_hbm_peak" % how: round(step_bytes / (ms / steps * 1e-3) / 1e9 / hbm, 4)}
+            out["kernels_per_step"] = dec.stats()[1]
+            dec.close()
+            del dec
+            torch.cuda.empty_cache()
+            rows.append(out)
+            print(json.dumps(out), file=sys.stderr, flush=True)
+    clocks = sampler.finish()
+    print(json.dumps({"compare": "dekalorn vs %s (bf16, random weights, synthetic tokens)" % args.compare_models, "rows": rows,
+                      "clocks": clocks, "timing": "CUDA events on the model's stream; weights per pass larger than L2"}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -839,6 +968,8 @@ def main():
                     help="instead of the default workload: Lagelorn beside Kodupel at a few layer sizes")
     ap.add_argument("--compare-dizizen", action="store_true",
                     help="instead of the default workload: Dizizen beside Kodupel at a few layer sizes")
+    ap.add_argument("--compare-dekalorn", action="store_true",
+                    help="instead of the default workload: Dekalorn beside Kodupel at a few layer sizes")
     ap.add_argument("--compare-dekipel", action="store_true",
                     help="instead of the default workload: Dekipel beside the bf16 Llama decoder at a few layer sizes")
     args = ap.parse_args()
@@ -849,6 +980,11 @@ def main():
         if args.compare_models == "dekipel,llama":
             args.compare_models = "dizizen,kodupel"
         run_compare_dizizen(args)
+        return
+    if args.compare_dekalorn:
+        if args.compare_models == "dekipel,llama":
+            args.compare_models = "dekalorn,kodupel"
+        run_compare_dekalorn(args)
         return
     if args.compare_lagelorn:
         if args.compare_models == "dekipel,llama":

@@ -793,3 +793,122 @@ def gated_parallel_combine(x, mult, gates, ga_off, a, scale_a, eps, parts=None, 
               _p(coef), _p(choice), n_parts, n_real, _p(f_dense), d, gf_off, _p(scale_f), _p(norm_w), _p(next_w), _p(h),
               _dt(h) if h is not None else F32, t, d, eps, 0, _stream())
     return h
+
+
+# ------------------------------------------------------------------ pre-norm residual, window attention with two maps, mixed
+# heads, latents with a rotated key part, routing by the two best of a group
+GEMM_EPI_REGLU = 8
+MOE_GROUP_MAX, MOE_GROUP_TOP2 = 0, 1
+
+
+def gemm_nt_reglu(x, w, out_dtype=None):
+    """y (M, N / 2) = max(gate, 0) * up over the column pairs (gate, up) of x @ w^T; w (N, K) with gate / up rows interleaved."""
+    m, k = x.shape
+    n = w.shape[0]
+    y = torch.empty((m, n // 2), dtype=out_dtype or x.dtype, device=x.device)
+    _lib.call("zl_gemm_nt_fused", _p(x), k, _p(w), k, None, _p(y), n // 2, m, n, k, _dt(x), _dt(y), GEMM_EPI_REGLU, None, 0, 0.0, 0,
+              _stream())
+    return y
+
+
+def moe_route_ex(x, w_router, top, groups=1, keep=1, group_rank=MOE_GROUP_TOP2, correction=None, score_fn=MOE_SCORE_SIGMOID,
+                 renormalize=True, renorm_eps=0.0, weight_scale=1.0):
+    """moe_route_grouped with x (T, D) and w_router (E, D) of one dtype (fp32 or 16-bit), the groups ranked by their largest
+    or the sum of their two largest scores, and the weights times weight_scale."""
+    t, d = x.shape
+    e = w_router.shape[0]
+    dev = x.device
+    te = torch.empty((t, top), dtype=torch.int32, device=dev)
+    tw = torch.empty((t, top), dtype=torch.float32, device=dev)
+    off = torch.empty(e + 1, dtype=torch.int32, device=dev)
+    lt = torch.empty(t * top, dtype=torch.int32, device=dev)
+    lp = torch.empty(t * top, dtype=torch.int32, device=dev)
+    _lib.call("zl_moe_route_ex", _p(x), d, _p(w_router), _dt(x), _p(correction), _p(te), _p(tw), _p(off), _p(lt), _p(lp), t, d, e, top,
+              groups, keep, group_rank, score_fn, int(renormalize), renorm_eps, weight_scale, 0, _stream())
+    return te, tw, off, lt, lp
+
+
+def residual_norm(x, parts=None, coef=None, next_w=None, x_copy=None, eps=1e-6, act_dtype=torch.float32):
+    """x (T, D) fp32 += sum_p coef[:, p] * parts[:, p] (parts (T, P, D) fp32) in place; x_copy (T, >= D) of act_dtype receives the
+    new x in its first D columns; returns next_w * rms(new x) in act_dtype when next_w is given."""
+    t, d = x.shape
+    h = torch.empty((t, d), dtype=act_dtype, device=x.device) if next_w is not None else None
+    _lib.call("zl_residual_norm", _p(x), d, _p(parts), d, _p(coef), parts.shape[1] if parts is not None else 0, _p(next_w), _p(h),
+              _p(x_copy), x_copy.shape[1] if x_copy is not None else 0, {torch.float16: F16, torch.bfloat16: BF16, torch.float32: F32}[act_dtype], t, d, eps, 0, _stream())
+    return h
+
+
+def embed_norm(ids, table, next_w=None, x_copy=None, x_copy2=None, eps=1e-6):
+    """ids (T) int32, table (V, D) -> (x (T, D) fp32, next_w * rms(x) in the table's dtype or None); the copies (views into
+    rows of one width) receive x in the table's dtype."""
+    t, d = ids.numel(), table.shape[1]
+    x = torch.empty((t, d), dtype=torch.float32, device=table.device)
+    h = torch.empty((t, d), dtype=table.dtype, device=table.device) if next_w is not None else None
+    views = [c.data_ptr() if c is not None else None for c in (x_copy, x_copy2)]
+    ld = max((c.stride(0) for c in (x_copy, x_copy2) if c is not None), default=0)
+    _lib.call("zl_embed_norm", _p(ids), _p(table), table.shape[0], _p(x), _p(next_w), _p(h), views[0], views[1], ld, _dt(table), t, d,
+              eps, 0, _stream())
+    return x, h
+
+
+def rope_inv_freq_wavelength(base, dims, scaling=None):
+    """numpy float64 (dims / 2): base^(-2i/dims), scaled by wavelength with scaling = (factor, low, high, original)."""
+    import numpy as np
+    out = np.zeros(dims // 2, dtype=np.float64)
+    factor, low, high, original = scaling or (0.0, 0.0, 0.0, 0.0)
+    _lib.call("zl_rope_inv_freq_wavelength", float(base), dims, float(factor), float(low), float(high), float(original),
+              out.ctypes.data_as(ctypes.POINTER(ctypes.c_double)))
+    return out
+
+
+def window_attention(q, k_table, v_table, slot, pos, scale, window, heads, kv_heads, dim, vdim, maps=1, lam=0.0, out_eps=0.0,
+                     out_mul=1.0, gate=None, splits=1, run_row0=None, run_len=None, max_run_len=0):
+    """Sliding-window attention; maps = 2: differential attention (q (T, heads * 2 * dim), keys of 2 * dim per head), gate
+    (T, heads * vdim) fp32 logits or None.  -> (T, heads * vdim) of q's dtype."""
+    t = q.shape[0]
+    nbytes = _lib.load().zl_sink_attention_workspace_bytes(t, heads * maps, vdim, splits)
+    ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=q.device)
+    out = torch.empty((t, heads * vdim), dtype=q.dtype, device=q.device)
+    _lib.call("zl_window_attention", _p(q), _p(k_table), _p(v_table), _p(slot), _p(pos), scale, window, maps, lam, out_eps, out_mul,
+              _p(gate), gate.shape[1] if gate is not None else 0, _p(out), t, heads, kv_heads, dim, vdim, splits, _p(ws), nbytes,
+              _p(run_row0), _p(run_len), run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(q), 0, _stream())
+    return out
+
+
+def mixed_head_attention(q, k_table, v_table, slot, pos, mix, window, heads, kv_heads, dim, vdim, splits=1, run_row0=None,
+                         run_len=None, max_run_len=0):
+    """Attention whose heads' scores are mixed by mix (heads, heads) fp32 (the scale folded in) before the softmax."""
+    t = q.shape[0]
+    nbytes = _lib.load().zl_sink_attention_workspace_bytes(t, heads, vdim, splits)
+    ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=q.device)
+    out = torch.empty((t, heads * vdim), dtype=q.dtype, device=q.device)
+    _lib.call("zl_mixed_head_attention", _p(q), _p(k_table), _p(v_table), _p(slot), _p(pos), _p(mix), window, _p(out), t, heads,
+              kv_heads, dim, vdim, splits, _p(ws), nbytes, _p(run_row0), _p(run_len),
+              run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(q), 0, _stream())
+    return out
+
+
+def latent_rope_append(proj, q_off, heads, dim, rot_dim, table, c_off, kv_rank, kv_weight, rank_cols, qa, cache, slot_tab, slot, pos,
+                       eps):
+    """-> q (T, heads, dim) unrotated query parts of the cache's dtype; qa (T, heads, row_cols) fp32 receives the rotated parts
+    behind its first rank_cols columns, cache (slots, rows, row_cols) the normed latent and the rotated key part."""
+    t, ldp = proj.shape
+    q = torch.empty((t, heads, dim), dtype=cache.dtype, device=proj.device)
+    _lib.call("zl_latent_rope_append", _p(proj), ldp, q_off, heads, dim, rot_dim, _p(table), _p(q), _p(qa), c_off, kv_rank,
+              _p(kv_weight), rank_cols, cache.shape[2], _p(slot_tab), _p(slot), _p(pos), t, eps, _dt(cache), 0, _stream())
+    return q
+
+
+def latent_attention_ex(q_absorbed, cache, table, slot, pos, scale, rank_cols, sink=None, gate=None, splits=1):
+    """q_absorbed (T, H, row_cols) fp32, cache (slots, rows, row_cols): all columns score, the first rank_cols are the value
+    -> (T, H, rank_cols) of the cache dtype; sink (H) or None, gate (T, H) fp32 logits or None."""
+    t, h, rs = q_absorbed.shape
+    lib = _lib.load()
+    _lib.check(lib.zl_latent_attention_prepare_ex(h, rank_cols, rs, _dt(cache)))
+    nbytes = lib.zl_latent_attention_workspace_bytes(t, h, rank_cols, splits)
+    ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=cache.device)
+    out = torch.empty((t, h, rank_cols), dtype=cache.dtype, device=cache.device)
+    _lib.call("zl_latent_attention_ex", _p(q_absorbed), _p(table), _p(slot), _p(pos), _p(sink), _p(gate),
+              gate.shape[1] if gate is not None else 0, scale, _p(out), t, h, rank_cols, rs, splits, _p(ws), nbytes, _dt(cache), 0,
+              _stream())
+    return out
