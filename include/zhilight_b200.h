@@ -755,11 +755,13 @@ int zl_latent_rope_append(const float* proj, long long ldp, int q_off, int heads
 /* zl_latent_attention over rows of row_cols columns of which all enter the score and the first rank_cols are the value:
  * q_absorbed (T, heads, row_cols) fp32, out (T, heads, rank_cols) of `dtype`.  sink NULL: an ordinary softmax.
  * gate != NULL: head h's output times sigmoid(gate[t * ldg + h]).  The probabilities enter the 16-bit product as a hi + lo
- * pair.  Workspace and splits as for kv_rank = rank_cols. */
+ * pair.  With the runs of the step (as in zl_sink_attention; run_row0 NULL: none) prompts take 64-row tiles of a run's tokens
+ * and heads.  Workspace and splits as for kv_rank = rank_cols. */
 int zl_latent_attention_prepare_ex(int heads, int rank_cols, int row_cols, int dtype);
 int zl_latent_attention_ex(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
                            const float* sink, const float* gate, long long ldg, float scale, void* out, int T, int heads,
-                           int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes, int dtype, int pdl,
+                           int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
+                           const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
                            zl_stream_t stream);
 /* ------------------------------------------------------------------------------------------ *
  * Kodupel: decoder-only model whose layers are listed one by one: the mixer is attention (grouped key/value heads,

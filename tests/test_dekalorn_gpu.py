@@ -355,6 +355,20 @@ def test_latent_attention_with_rotated_part(cuda, lib, dtype, shape):
                                               gate=dev(gate[rows], cuda) if g else None, splits=splits).float().cpu().numpy()
                 ref = want * orc.sigmoid(gate[rows].astype(np.float64))[:, :, None] if g else want
                 assert np.abs(out[:, :, :R] - ref).max() < tol and np.abs(out[:, :, R:]).max(initial=0.0) == 0.0, (splits, g, use_sink)
+    # two runs of consecutive tokens: the tiles of a prompt
+    seq = list(range(5)) + list(range(230, 300))
+    s = np.einsum("thc,jc->thj", qa[seq].astype(np.float64), c.astype(np.float64)) * scale
+    for use_sink in (False, True):
+        want = np.zeros((len(seq), H, R))
+        for i, t in enumerate(seq):
+            e = np.exp(s[i, :, :t + 1])
+            want[i] = e @ c[:t + 1, :R] / (e.sum(-1, keepdims=True) + (np.exp(sink)[:, None] if use_sink else 0.0))
+        want *= orc.sigmoid(gate[seq].astype(np.float64))[:, :, None]
+        for splits in (1, 3):
+            out = ops.latent_attention_ex(dev(qa[seq], cuda), cache, ops.slot_table(cache), i32([1] * len(seq), cuda), i32(seq, cuda), scale,
+                                          RC, sink=dev(sink, cuda) if use_sink else None, gate=dev(gate[seq], cuda), splits=splits,
+                                          **_runs(cuda, [5, 70])).float().cpu().numpy()
+            assert np.abs(out[:, :, :R] - want).max() < tol and np.abs(out[:, :, R:]).max(initial=0.0) == 0.0, (splits, use_sink, "runs")
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

@@ -392,7 +392,8 @@ int enqueue_mixer(zl_dekalorn* m, KRun& U, int T, int n_runs, int max_run, int m
         RCHECK(zl_gemm_nt(m->q, (long long)H * d, d, L.uk_t, d, (long long)RC * d, m->qa, (long long)H * RS, RS, T, RC, d, H, dt, ZL_F32,
                           ZL_GEMM_EPI_NONE, nullptr, 0, 0, pg, st));
         RCHECK(zl_latent_attention_ex(m->qa, U.a.addrs, m->d_slots, m->d_pos, nullptr, m->proj + L.g_off, L.n_in, lc.scale, m->olat, T, H,
-                                      RC, RS, splits, m->attn_ws, m->attn_ws_bytes, dt, pa, st));
+                                      RC, RS, splits, m->attn_ws, m->attn_ws_bytes, m->d_run0, m->d_runlen, n_runs, max_run, dt, pa,
+                                      st));
         RCHECK(zl_gemm_nt(m->olat, (long long)H * RC, RC, L.uv, RC, (long long)vd * RC, m->att, (long long)H * vd, vd, T, vd, RC, H, dt,
                           dt, ZL_GEMM_EPI_NONE, nullptr, 0, 0, pg, st));
     } else if (lc.type == ZL_DEKALORN_DIFF) {

@@ -179,7 +179,9 @@ __global__ void k_latent_attn_merge(const float* __restrict__ part_acc, const fl
 // enter the MMAs as bfloat16.
 constexpr int kLmKeys = 32;
 constexpr int kLmRows = 16;
-constexpr int kLmStages = 3;   // latent tiles in flight per CTA
+// latent tiles in flight per CTA; the general form's longer rows leave room for two if two CTAs are to share an SM
+template <bool EX>
+constexpr int lm_stages() { return EX ? 2 : 3; }
 
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
     __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
@@ -191,6 +193,11 @@ __device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc) {
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem_row) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"(smem_u32(smem_row)));
+}
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* smem_row) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
@@ -205,7 +212,8 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
     const int RS = EX ? p.RS : R, RP = RS + 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* sc = reinterpret_cast<__nv_bfloat16*>(smem_raw);                       // [stages][32][RP]
-    float* ss = reinterpret_cast<float*>(smem_raw + (size_t)kLmStages * kLmKeys * RP * 2);   // [4][16][34]
+    constexpr int STG = lm_stages<EX>();
+    float* ss = reinterpret_cast<float*>(smem_raw + (size_t)STG * kLmKeys * RP * 2);   // [4][16][34]
     pdl_trigger();
     pdl_wait();
     const int h0 = blockIdx.x * kLmRows, t = blockIdx.y, split = blockIdx.z;
@@ -268,14 +276,16 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
         cp_async_commit();
     };
     const int n_tiles = hi > lo ? cdiv(hi - lo, kLmKeys) : 0;
-    if (n_tiles > 0) stage(lo, 0);
-    if (n_tiles > 1) stage(lo + kLmKeys, 1);
-    else cp_async_commit();
+#pragma unroll
+    for (int i = 0; i < STG - 1; ++i) {
+        if (i < n_tiles) stage(lo + i * kLmKeys, i);
+        else cp_async_commit();
+    }
     for (int it = 0; it < n_tiles; ++it) {
-        const int j0 = lo + it * kLmKeys, buf = it % kLmStages;
-        cp_async_wait<1>();   // all but the youngest group: tile `it` has landed
+        const int j0 = lo + it * kLmKeys, buf = it % STG;
+        cp_async_wait<STG - 2>();   // all but the younger groups: tile `it` has landed
         __syncthreads();      // ... for every thread; every warp is done with round it - 1 (its buffer, the score tiles)
-        if (it + 2 < n_tiles) stage(j0 + 2 * kLmKeys, (it + 2) % kLmStages);   // two tiles ahead of the math
+        if (it + STG - 1 < n_tiles) stage(j0 + (STG - 1) * kLmKeys, (it + STG - 1) % STG);   // ahead of the math
         else cp_async_commit();
         const __nv_bfloat16* ct = sc + (size_t)buf * kLmKeys * RP;
         // partial scores over this warp's quarter of kv_rank
@@ -395,14 +405,221 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
     }
 }
 
+// ---- prompt form of the general tensor-core kernel ---------------------------------------------------------------------
+// One CTA = 64 rows = (consecutive tokens of one run) x (heads), one key range; 8 warps in pairs of the same 16 rows.  Every
+// 32-key latent tile serves all 64 rows (cp.async, two tiles in flight; the queries stay in shared memory).  S: a warp takes
+// 16 of the 32 keys over the whole contraction; the pair exchanges its score halves through shared memory; both warps then
+// hold the same softmax state, and each owns half of the value columns of O += P C.
+constexpr int kLtRows = 64, kLtKeys = 32, kLtStages = 2, kLtSp = kLtKeys + 4;
+
+struct LaTileP {
+    LaParams<__nv_bfloat16> a;
+    const int32_t *run_row0, *run_len;
+    int hb, nq;   // heads and tokens per tile
+};
+
+template <int NK>
+__global__ void __launch_bounds__(256, 1) k_latent_tile_mma(LaTileP pp) {
+    constexpr int R = 64 * NK, NT = 4 * NK;   // value columns; 8-column tiles per warp
+    const LaParams<__nv_bfloat16>& p = pp.a;
+    const int RS = p.RS, RP = RS + 8, H = p.H;
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw);          // [64][RP]
+    __nv_bfloat16* sc = sq + (size_t)kLtRows * RP;                           // [stages][32][RP]
+    float* ss = reinterpret_cast<float*>(sc + (size_t)kLtStages * kLtKeys * RP);   // [64][kLtSp]
+    pdl_trigger();
+    pdl_wait();
+    const int run = blockIdx.z / p.S, split = blockIdx.z - run * p.S, h0 = blockIdx.x * pp.hb;
+    const int len = pp.run_len[run], t0 = (int)(gridDim.y - 1 - blockIdx.y) * pp.nq;   // the tiles with the most keys start first
+    if (t0 >= len) return;
+    const int ntok = min(pp.nq, len - t0), row0 = pp.run_row0[run] + t0, hb = pp.hb, hn = min(hb, H - h0);
+    const int pos0 = p.pos[row0];
+    const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.slot_addrs[p.slot[row0]]);
+    int lo = 0, hi = pos0 + ntok;
+    if (p.S > 1) {
+        const int per = cdiv(cdiv(hi, p.S), kLtKeys) * kLtKeys;
+        lo = split * per;
+        hi = min(hi, lo + per);
+    }
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
+    const int rb = warp >> 1, hf = warp & 1;
+    const int n8 = RS / 8;
+    auto stage = [&](int j0, int buf) {   // keys past `hi` are zero rows
+        __nv_bfloat16* dst = sc + (size_t)buf * kLtKeys * RP;
+        for (int j = warp; j < kLtKeys; j += 8)
+            for (int c = lane; c < n8; c += 32) {
+                if (j0 + j < hi) cp_async16(dst + j * RP + c * 8, cache + (size_t)(j0 + j) * RS + c * 8);
+                else *reinterpret_cast<uint4*>(dst + j * RP + c * 8) = make_uint4(0, 0, 0, 0);
+            }
+        cp_async_commit();
+    };
+    int t_of[2], h_of[2], pos_of[2];
+    bool ok[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int r = rb * 16 + g + i * 8, tk = r / hb;
+        t_of[i] = row0 + tk;
+        h_of[i] = h0 + r - tk * hb;
+        ok[i] = tk < ntok && h_of[i] < H;
+        pos_of[i] = ok[i] ? pos0 + tk : -1;
+    }
+    float m_run[2], l_run[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const bool with_sink = p.S == 1 && p.sink && ok[i];
+        m_run[i] = with_sink ? p.sink[h_of[i]] : -INFINITY;
+        l_run[i] = with_sink ? 1.f : 0.f;
+    }
+    float o[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
+    const int n_tiles = hi > lo ? cdiv(hi - lo, kLtKeys) : 0;
+    if (n_tiles > 0) {
+        stage(lo, 0);
+        for (int r = warp; r < kLtRows; r += 8) {
+            const int tk = r / hb, h = r - tk * hb;
+            const bool in = tk < ntok && h < hn;
+            const float* src = p.qa + ((size_t)(row0 + (in ? tk : 0)) * H + h0 + (in ? h : 0)) * RS;
+            for (int c = lane; c < RS / 4; c += 32) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (in) v = reinterpret_cast<const float4*>(src)[c];
+                *reinterpret_cast<uint2*>(sq + (size_t)r * RP + c * 4) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+            }
+        }
+    }
+    for (int it = 0; it < n_tiles; ++it) {
+        const int j0 = lo + it * kLtKeys;
+        cp_async_wait<0>();
+        __syncthreads();   // tile `it` (and the queries) are in place; every warp is done with the other buffer and the scores
+        if (it + 1 < n_tiles) stage(j0 + kLtKeys, (it + 1) & 1);
+        const __nv_bfloat16* ct = sc + (size_t)(it & 1) * kLtKeys * RP;
+        float s[4][4];   // two 8-key tiles, each in two chains over alternating contraction steps
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) s[i][c] = 0.f;
+        const __nv_bfloat16* qrow = sq + (size_t)(rb * 16 + (lane & 15)) * RP + (lane >> 4) * 8;
+        const __nv_bfloat16* krow = ct + (size_t)(hf * 16 + (lane & 7) + (lane >> 4) * 8) * RP + ((lane >> 3) & 1) * 8;
+#pragma unroll 4
+        for (int ks = 0; ks < RS / 16; ++ks) {
+            uint32_t a[4], b[4];
+            ldmatrix_x4(a, qrow + ks * 16);
+            ldmatrix_x4(b, krow + ks * 16);
+            if (ks & 1) {
+                mma_16816_bf16(s[2], a, b[0], b[1], s[2]);
+                mma_16816_bf16(s[3], a, b[2], b[3], s[3]);
+            } else {
+                mma_16816_bf16(s[0], a, b[0], b[1], s[0]);
+                mma_16816_bf16(s[1], a, b[2], b[3], s[1]);
+            }
+        }
+        float* sr = ss + (size_t)rb * 16 * kLtSp;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            float* d = sr + (size_t)g * kLtSp + hf * 16 + i * 8 + 2 * q4;
+            *reinterpret_cast<float2*>(d) = make_float2(s[i][0] + s[i + 2][0], s[i][1] + s[i + 2][1]);
+            *reinterpret_cast<float2*>(d + 8 * kLtSp) = make_float2(s[i][2] + s[i + 2][2], s[i][3] + s[i + 2][3]);
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(1 + rb) : "memory");   // the pair's halves are in place
+        float v[4][4], mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const float2 x = *reinterpret_cast<const float2*>(sr + (size_t)(g + i * 8) * kLtSp + nt * 8 + 2 * q4);
+                const int j = j0 + nt * 8 + 2 * q4;
+                v[nt][2 * i] = j < hi && j <= pos_of[i] ? x.x * p.scale : -INFINITY;
+                v[nt][2 * i + 1] = j + 1 < hi && j + 1 <= pos_of[i] ? x.y * p.scale : -INFINITY;
+                mx[i] = fmaxf(mx[i], fmaxf(v[nt][2 * i], v[nt][2 * i + 1]));
+            }
+        float corr[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+            const float m_new = fmaxf(m_run[i], mx[i]), m_use = m_new == -INFINITY ? 0.f : m_new;
+            corr[i] = expf(m_run[i] - m_use);
+            m_run[i] = m_new;
+            mx[i] = m_use;
+        }
+        uint32_t ph[2][4], pl[2][4];
+        auto rest = [](float x) { return x - __bfloat162float(__float2bfloat16_rn(x)); };
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const float x = expf(v[nt][2 * i] - mx[i]), y = expf(v[nt][2 * i + 1] - mx[i]);
+                sum[i] += x + y;
+                ph[nt >> 1][(nt & 1) * 2 + i] = pack_bf16(x, y);
+                pl[nt >> 1][(nt & 1) * 2 + i] = pack_bf16(rest(x), rest(y));
+            }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+            sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+            l_run[i] = l_run[i] * corr[i] + sum[i];
+        }
+        if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) o[nt][0] *= corr[0], o[nt][1] *= corr[0], o[nt][2] *= corr[1], o[nt][3] *= corr[1];
+        }
+        const __nv_bfloat16* vrow = ct + (size_t)lane * RP + hf * (R / 2);
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+            uint32_t bv[4];
+            ldmatrix_x4_trans(bv, vrow + nt * 8);
+            mma_16816_bf16(o[nt], ph[0], bv[0], bv[1], o[nt]);
+            mma_16816_bf16(o[nt], ph[1], bv[2], bv[3], o[nt]);
+            mma_16816_bf16(o[nt], pl[0], bv[0], bv[1], o[nt]);
+            mma_16816_bf16(o[nt], pl[1], bv[2], bv[3], o[nt]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        if (!ok[i]) continue;
+        const size_t th = (size_t)t_of[i] * H + h_of[i];
+        const float f = p.S > 1 ? 1.f : la_gate(p.gate, p.ldg, t_of[i], h_of[i]) / l_run[i];
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+            const int col = hf * (R / 2) + nt * 8 + 2 * q4;
+            if (p.S > 1)
+                *reinterpret_cast<float2*>(p.part_acc + (th * p.S + split) * R + col) = make_float2(o[nt][2 * i], o[nt][2 * i + 1]);
+            else
+                *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + th * R + col) = pack_bf16(o[nt][2 * i] * f, o[nt][2 * i + 1] * f);
+        }
+        if (p.S > 1 && hf == 0 && q4 == 0) {
+            p.part_ml[(th * p.S + split) * 2] = m_run[i];
+            p.part_ml[(th * p.S + split) * 2 + 1] = l_run[i];
+        }
+    }
+}
+
+static size_t lt_smem_bytes(int RS) {
+    return ((size_t)kLtRows + (size_t)kLtStages * kLtKeys) * (RS + 8) * 2 + (size_t)kLtRows * kLtSp * 4;
+}
+template <int NK>
+static cudaError_t lt_launch(const LaTileP& pp, dim3 grid, bool pdl, cudaStream_t st) {
+    const size_t smem = lt_smem_bytes(pp.a.RS);
+    static size_t set_for = 0;
+    if (smem > 48 * 1024 && smem > set_for) {
+        const cudaError_t e = cudaFuncSetAttribute(k_latent_tile_mma<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+        set_for = smem;
+    }
+    return launch(k_latent_tile_mma<NK>, grid, dim3(256), smem, st, pdl, pp);
+}
+
 static bool lm_eligible(int dtype, int R) {
     static const bool off = getenv("ZL_LATENT_ATTN_NO_MMA") != nullptr;
     return !off && dtype == ZL_BF16 && R % 64 == 0 && R >= 64 && R <= 512;
 }
-static size_t lm_smem_bytes(int RS) { return (size_t)kLmStages * kLmKeys * (RS + 8) * 2 + (size_t)4 * kLmRows * 34 * 4; }
+template <bool EX>
+static size_t lm_smem_bytes(int RS) { return (size_t)lm_stages<EX>() * kLmKeys * (RS + 8) * 2 + (size_t)4 * kLmRows * 34 * 4; }
 // the general form needs its score-only columns in whole 16-column steps, at most one per warp
 static bool lm_eligible_ex(int dtype, int R, int RS) {
-    return lm_eligible(dtype, R) && (RS - R) % 16 == 0 && RS - R <= 64 && lm_smem_bytes(RS) <= 200 * 1024;
+    return lm_eligible(dtype, R) && (RS - R) % 16 == 0 && RS - R <= 64 && lm_smem_bytes<true>(RS) <= 200 * 1024;
 }
 
 template <int NK, bool EX>
@@ -415,7 +632,7 @@ static cudaError_t lm_attr(int bytes) {   // the largest request stands: models 
 }
 template <bool EX>
 static cudaError_t lm_prepare(int R, int RS) {
-    const int b = (int)lm_smem_bytes(RS);
+    const int b = (int)lm_smem_bytes<EX>(RS);
     switch (R / 64) {
         case 1: return lm_attr<1, EX>(b);
         case 2: return lm_attr<2, EX>(b);
@@ -430,7 +647,7 @@ static cudaError_t lm_prepare(int R, int RS) {
 
 template <bool EX>
 static int lm_launch(const LaParams<__nv_bfloat16>& p, int T, bool pdl, cudaStream_t st) {
-    const size_t smem = lm_smem_bytes(p.RS);
+    const size_t smem = lm_smem_bytes<EX>(p.RS);
     const dim3 grid(cdiv(p.H, kLmRows), T, p.S), block(128);
     switch (p.R / 64) {
         case 1: ZL_CHECK_CUDA(launch(k_latent_attn_mma<1, EX>, grid, block, smem, st, pdl, p)); break;
@@ -441,6 +658,28 @@ static int lm_launch(const LaParams<__nv_bfloat16>& p, int T, bool pdl, cudaStre
         case 6: ZL_CHECK_CUDA(launch(k_latent_attn_mma<6, EX>, grid, block, smem, st, pdl, p)); break;
         case 7: ZL_CHECK_CUDA(launch(k_latent_attn_mma<7, EX>, grid, block, smem, st, pdl, p)); break;
         default: ZL_CHECK_CUDA(launch(k_latent_attn_mma<8, EX>, grid, block, smem, st, pdl, p)); break;
+    }
+    if (p.S > 1)
+        ZL_CHECK_CUDA(launch(k_latent_attn_merge<__nv_bfloat16>, dim3(p.H, T), dim3(128), 0, st, pdl, (const float*)p.part_acc,
+                             (const float*)p.part_ml, p.sink, p.gate, p.ldg, static_cast<__nv_bfloat16*>(p.out), p.H, p.R, p.S));
+    return ZL_OK;
+}
+
+// the prompt form: tiles of 64 rows over the runs of the step
+static int lt_run(const LaParams<__nv_bfloat16>& p, const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int T,
+                  bool pdl, cudaStream_t st) {
+    const int hb = p.H < kLtRows ? p.H : kLtRows, nq = kLtRows / hb;
+    const LaTileP pp{p, run_row0, run_len, hb, nq};
+    const dim3 grid(cdiv(p.H, hb), cdiv(max_run_len, nq), runs * p.S);
+    switch (p.R / 64) {
+        case 1: ZL_CHECK_CUDA(lt_launch<1>(pp, grid, pdl, st)); break;
+        case 2: ZL_CHECK_CUDA(lt_launch<2>(pp, grid, pdl, st)); break;
+        case 3: ZL_CHECK_CUDA(lt_launch<3>(pp, grid, pdl, st)); break;
+        case 4: ZL_CHECK_CUDA(lt_launch<4>(pp, grid, pdl, st)); break;
+        case 5: ZL_CHECK_CUDA(lt_launch<5>(pp, grid, pdl, st)); break;
+        case 6: ZL_CHECK_CUDA(lt_launch<6>(pp, grid, pdl, st)); break;
+        case 7: ZL_CHECK_CUDA(lt_launch<7>(pp, grid, pdl, st)); break;
+        default: ZL_CHECK_CUDA(lt_launch<8>(pp, grid, pdl, st)); break;
     }
     if (p.S > 1)
         ZL_CHECK_CUDA(launch(k_latent_attn_merge<__nv_bfloat16>, dim3(p.H, T), dim3(128), 0, st, pdl, (const float*)p.part_acc,
@@ -503,6 +742,7 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
     if (unit < p.H) {
         const float* src = row + p.q_off + (size_t)unit * (p.d + p.rd);
         TO* dst = static_cast<TO*>(p.q_out) + ((size_t)t * p.H + unit) * p.d;
+#pragma unroll 4
         for (int c = lane; c < p.d; c += 32) dst[c] = from_f32<TO>(src[c]);
         float* qr = p.qa + ((size_t)t * p.H + unit) * p.row_cols + p.rank_cols;
         for (int i = lane; i < (p.rd >> 1); i += 32) {
@@ -524,10 +764,23 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
         }
         return;
     }
-    float ss = 0.f;
-    for (int c = lane; c < p.R; c += 32) ss = fmaf(src[c], src[c], ss);
+    float keep[16], wv[16], ss = 0.f;   // the first 512 columns in registers, every load in flight at once
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int c = lane + 32 * i;
+        keep[i] = c < p.R ? src[c] : 0.f;
+        wv[i] = c < p.R ? p.kv_w[c] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) ss = fmaf(keep[i], keep[i], ss);
+    for (int c = lane + 512; c < p.R; c += 32) ss = fmaf(src[c], src[c], ss);
     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)p.R + p.eps);
-    for (int c = lane; c < p.R; c += 32) dst[c] = from_f32<TO>(src[c] * r * p.kv_w[c]);
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int c = lane + 32 * i;
+        if (c < p.R) dst[c] = from_f32<TO>(keep[i] * r * wv[i]);
+    }
+    for (int c = lane + 512; c < p.R; c += 32) dst[c] = from_f32<TO>(src[c] * r * p.kv_w[c]);
 }
 
 }  // namespace zl
@@ -602,13 +855,14 @@ extern "C" int zl_latent_attention(const float* q_absorbed, void* const* slot_ad
         return lm_launch<false>(la_params<__nv_bfloat16>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, kv_rank, kv_rank,
                                                          splits, workspace, nullptr, 0), T, pdl != 0, stream);
     return zl_latent_attention_ex(q_absorbed, slot_addrs, slot, pos, sink, nullptr, 0, scale, out, T, heads, kv_rank, kv_rank, splits,
-                                  workspace, workspace_bytes, dtype, pdl, stream);
+                                  workspace, workspace_bytes, nullptr, nullptr, 0, 0, dtype, pdl, stream);
 }
 
 extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
                                       const float* sink, const float* gate, long long ldg, float scale, void* out, int T,
                                       int heads, int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
-                                      int dtype, int pdl, zl_stream_t stream) {
+                                      const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
+                                      zl_stream_t stream) {
     ZL_CHECK_ARG(q_absorbed && slot_addrs && slot && pos && out && T > 0 && T <= 65535 && heads > 0 && rank_cols > 0);
     ZL_CHECK_ARG(row_cols >= rank_cols && (dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32));
     ZL_CHECK_ARG(splits >= 1 && splits <= 64 && heads <= 65535);
@@ -619,7 +873,13 @@ extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot
     la_params<TC>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, rank_cols, row_cols, splits, workspace, gate, ldg)
     if (dtype == ZL_F32) return la_launch<float>(ZL_LA_P(float), T, pdl != 0, stream);
     if (dtype == ZL_F16) return la_launch<__half>(ZL_LA_P(__half), T, pdl != 0, stream);
-    if (lm_eligible_ex(dtype, rank_cols, row_cols) && row_cols % 8 == 0 && (reinterpret_cast<uintptr_t>(q_absorbed) & 7) == 0)
+    const bool mma = lm_eligible_ex(dtype, rank_cols, row_cols) && row_cols % 8 == 0 && (reinterpret_cast<uintptr_t>(q_absorbed) & 15) == 0;
+    // runs whose rows fill more than one 16-row tile per key tile: a prompt
+    static const bool no_tile = getenv("ZL_LATENT_ATTN_NO_TILE") != nullptr;
+    if (mma && !no_tile && run_row0 && run_len && runs > 0 && (long long)max_run_len * heads >= 2 * kLmRows && max_run_len > 1 &&
+        (long long)runs * splits <= 65535 && lt_smem_bytes(row_cols) <= 225 * 1024)
+        return lt_run(ZL_LA_P(__nv_bfloat16), run_row0, run_len, runs, max_run_len, T, pdl != 0, stream);
+    if (mma)
         return lm_launch<true>(ZL_LA_P(__nv_bfloat16), T, pdl != 0, stream);
     return la_launch<__nv_bfloat16>(ZL_LA_P(__nv_bfloat16), T, pdl != 0, stream);
 #undef ZL_LA_P

@@ -42,12 +42,22 @@ template <typename T>
 __device__ __forceinline__ float route_dot16(const T* __restrict__ a, const T* __restrict__ b, int D, int lane, bool vec) {
     float acc0 = 0.f, acc1 = 0.f;
     if (vec) {
-        for (int c = lane; c < (D >> 3); c += 32) {
-            float x[8], y[8];
-            unpack8<T>(reinterpret_cast<const uint4*>(a)[c], x);
-            unpack8<T>(reinterpret_cast<const uint4*>(b)[c], y);
+        const uint4 *a8 = reinterpret_cast<const uint4*>(a), *b8 = reinterpret_cast<const uint4*>(b);
+        const int n8 = D >> 3;
+        for (int c0 = lane; c0 < n8; c0 += 128) {   // four pieces of both rows in flight
+            uint4 u[4], v[4];
 #pragma unroll
-            for (int i = 0; i < 8; i += 2) acc0 = fmaf(x[i], y[i], acc0), acc1 = fmaf(x[i + 1], y[i + 1], acc1);
+            for (int k = 0; k < 4; ++k)
+                if (c0 + 32 * k < n8) u[k] = a8[c0 + 32 * k], v[k] = b8[c0 + 32 * k];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                if (c0 + 32 * k >= n8) break;
+                float x[8], y[8];
+                unpack8<T>(u[k], x);
+                unpack8<T>(v[k], y);
+#pragma unroll
+                for (int i = 0; i < 8; i += 2) acc0 = fmaf(x[i], y[i], acc0), acc1 = fmaf(x[i + 1], y[i + 1], acc1);
+            }
         }
     } else {
         for (int c = lane; c < D; c += 32) acc0 = fmaf(to_f32<T>(a[c]), to_f32<T>(b[c]), acc0);

@@ -677,19 +677,19 @@ __global__ void __launch_bounds__(128) k_sink_attn_merge(SinkAttnP p) {
     }
 }
 
-// the same for two maps per head: both maps' merged results meet, then the norm over the head and the gate
+// The same for two maps per head: a warp per map (two heads per CTA); the second map's merged sum goes through shared
+// memory to the first one's warp, which takes the difference, the norm over the head and the gate.
 template <typename T>
 __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
+    __shared__ float second[2][32 * kSaMaxPerLane];
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.y, h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (h >= p.H) return;
+    const int t = blockIdx.y, w = threadIdx.x >> 5, lane = threadIdx.x & 31, map = w & 1, h = blockIdx.x * 2 + (w >> 1);
+    const bool live = h < p.H;
     const int stride = 2 + p.vd;
-    float keep[kSaMaxPerLane], ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < kSaMaxPerLane; ++i) keep[i] = 0.f;
-    for (int mp = 0; mp < 2; ++mp) {
-        const float* part = p.ws + (((size_t)t * p.H + h) * 2 + mp) * p.splits * stride;
+    float keep[kSaMaxPerLane];
+    if (live) {
+        const float* part = p.ws + (((size_t)t * p.H + h) * 2 + map) * p.splits * stride;
         const float ms = lane < p.splits ? part[(size_t)lane * stride] : -INFINITY;
         const float ls = lane < p.splits ? part[(size_t)lane * stride + 1] : 0.f;
         const float M = warp_max(ms);
@@ -698,10 +698,11 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
 #pragma unroll
         for (int s = 0; s < 32; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
         for (int s = 0; s < p.splits; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, wgt, s), L);
-        const float f = (mp ? -p.lambda : 1.0f) / L;
+        const float f = (map ? p.lambda : 1.0f) / L;
 #pragma unroll
         for (int i = 0; i < kSaMaxPerLane; ++i) {
             const int c = lane + 32 * i;
+            keep[i] = 0.f;
             if (c >= p.vd) continue;
             float v[32];
 #pragma unroll
@@ -709,11 +710,19 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
             float o = 0.f;
 #pragma unroll
             for (int s = 0; s < 32; ++s) o = fmaf(v[s], wv[s], o);
-            keep[i] = fmaf(o, f, keep[i]);
+            keep[i] = o * f;
+            if (map) second[w >> 1][c] = keep[i];
         }
     }
+    __syncthreads();
+    if (!live || map) return;
+    float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < kSaMaxPerLane; ++i) ss = fmaf(keep[i], keep[i], ss);
+    for (int i = 0; i < kSaMaxPerLane; ++i) {
+        const int c = lane + 32 * i;
+        if (c < p.vd) keep[i] -= second[w >> 1][c];
+        ss = fmaf(keep[i], keep[i], ss);
+    }
     const float mul = p.out_mul / sqrtf(warp_sum(ss) / (float)p.vd + p.out_eps);
     T* out = static_cast<T*>(p.out) + ((size_t)t * p.H + h) * p.vd;
 #pragma unroll
@@ -728,7 +737,7 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
 
 template <typename T>
 static cudaError_t sa_merge_t(const SinkAttnP& p, int maps, int T_, bool pdl, cudaStream_t st) {
-    const dim3 mg(cdiv(p.H, 4), T_), mb(128);
+    const dim3 mg(cdiv(p.H, maps == 2 ? 2 : 4), T_), mb(128);
     return maps == 2 ? launch(k_two_map_merge<T>, mg, mb, 0, st, pdl, p) : launch(k_sink_attn_merge<T>, mg, mb, 0, st, pdl, p);
 }
 int sink_attn_merge(const SinkAttnP& p, int maps, int T, int dtype, bool pdl, cudaStream_t st) {

@@ -899,7 +899,8 @@ def latent_rope_append(proj, q_off, heads, dim, rot_dim, table, c_off, kv_rank, 
     return q
 
 
-def latent_attention_ex(q_absorbed, cache, table, slot, pos, scale, rank_cols, sink=None, gate=None, splits=1):
+def latent_attention_ex(q_absorbed, cache, table, slot, pos, scale, rank_cols, sink=None, gate=None, splits=1, run_row0=None,
+                        run_len=None, max_run_len=0):
     """q_absorbed (T, H, row_cols) fp32, cache (slots, rows, row_cols): all columns score, the first rank_cols are the value
     -> (T, H, rank_cols) of the cache dtype; sink (H) or None, gate (T, H) fp32 logits or None."""
     t, h, rs = q_absorbed.shape
@@ -909,6 +910,6 @@ def latent_attention_ex(q_absorbed, cache, table, slot, pos, scale, rank_cols, s
     ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=cache.device)
     out = torch.empty((t, h, rank_cols), dtype=cache.dtype, device=cache.device)
     _lib.call("zl_latent_attention_ex", _p(q_absorbed), _p(table), _p(slot), _p(pos), _p(sink), _p(gate),
-              gate.shape[1] if gate is not None else 0, scale, _p(out), t, h, rank_cols, rs, splits, _p(ws), nbytes, _dt(cache), 0,
-              _stream())
+              gate.shape[1] if gate is not None else 0, scale, _p(out), t, h, rank_cols, rs, splits, _p(ws), nbytes, _p(run_row0),
+              _p(run_len), run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(cache), 0, _stream())
     return out
