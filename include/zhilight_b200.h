@@ -733,14 +733,15 @@ int zl_window_attention(const void* q, void* const* k_addrs, void* const* v_addr
                         long long ldg, void* out, int T, int heads, int kv_heads, int dim, int vdim, int splits,
                         void* workspace, size_t workspace_bytes, const int32_t* run_row0, const int32_t* run_len, int runs,
                         int max_run_len, int dtype, int pdl, zl_stream_t stream);
-/* Attention whose heads' scores are mixed before the softmax: s'_h = sum_g mix[h * heads + g] (q_g . k_{g / (heads / kv_heads)})
- * (mix fp32 (heads, heads), the scores' scale folded in), ordinary softmax of s'_h over the visible keys (window as above),
- * out[t][h] = sum_j p_j v_{h / (heads / kv_heads)}.  Same caches, splits (zl_mixed_head_attention_splits) and runs;
- * workspace of zl_sink_attention_workspace_bytes. */
-int zl_mixed_head_attention_splits(int T, int heads, int max_len);
+/* Attention whose heads' scores are mixed before the softmax:
+ * s'_h = sum_g mix[h * heads + g] factor[g] (q_g . k_{g / (heads / kv_heads)}) (mix fp32 (heads, heads), rounded to 16 bits in
+ * 16-bit runs like every weight; factor fp32 (heads), the scores' scale folded in), ordinary softmax of s'_h over the
+ * visible keys (window as above), out[t][h] = sum_j p_j v_{h / (heads / kv_heads)}.  Same caches, splits
+ * (zl_mixed_head_attention_splits; T rows in `runs` runs) and runs; workspace of zl_sink_attention_workspace_bytes. */
+int zl_mixed_head_attention_splits(int T, int runs, int heads, int kv_heads, int dim, int vdim, int max_len);
 int zl_mixed_head_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot, const int32_t* pos,
-                            const float* mix, int window, void* out, int T, int heads, int kv_heads, int dim, int vdim,
-                            int splits, void* workspace, size_t workspace_bytes, const int32_t* run_row0,
+                            const float* mix, const float* factor, int window, void* out, int T, int heads, int kv_heads,
+                            int dim, int vdim, int splits, void* workspace, size_t workspace_bytes, const int32_t* run_row0,
                             const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl, zl_stream_t stream);
 /* From a fused projection row proj[t] (fp32) to the operands of absorbed latent attention with a rotated part: query head h
  * (columns q_off + h * (dim + rot_dim)): its first `dim` columns -> q_out (T, heads, dim) of `dtype`, its last rot_dim ones

@@ -287,7 +287,8 @@ def test_attention_with_mixed_heads(cuda, lib, dtype, shape):
     temp, talk = 1 + 0.3 * rng.standard_normal(H), np.eye(H) + 0.5 * rng.standard_normal((H, H)) / math.sqrt(H)
     talk[0] = 0.0
     talk[0, H - 1] = 1.5                                            # head 0 scores by the last head's query and keys only
-    mix = (talk * temp[None, :] * scale).astype(np.float32)
+    talk = b16(talk).astype(np.float64)                             # a weight: exact in bfloat16
+    factor = (temp * scale).astype(np.float32)
     tol = 4e-5 if dtype == "float32" else 2e-2
     for window in (1, 31, 32, 33, 64, 0):
         q, k = q0.copy(), k0.copy()
@@ -304,7 +305,7 @@ def test_attention_with_mixed_heads(cuda, lib, dtype, shape):
 
         def run(rows, **kw):
             return ops.mixed_head_attention(dev(q[rows].reshape(len(rows), -1), cuda, td), *tabs, i32([1] * len(rows), cuda),
-                                            i32(rows, cuda), dev(mix, cuda), window, H, G, d, vd, **kw).float().cpu().numpy()
+                                            i32(rows, cuda), dev(talk.astype(np.float32), cuda), dev(factor, cuda), window, H, G, d, vd, **kw).float().cpu().numpy()
 
         rows = [0, 1, 15, 16, 17, 31, 32, 33, 63, 64, 65, 127, 249, 250, 251, 289]
         seq = list(range(9)) + list(range(200, 290))

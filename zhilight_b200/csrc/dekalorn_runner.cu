@@ -12,7 +12,7 @@
 //   differential:  [W_q; W_k; W_v; W_g] -> append -> two softmax maps per head in a sliding window, their difference, norm and
 //                  gate in one kernel (sink_attn.cu) -> W_o.
 //   mixed heads:   [W_q; W_k; W_v] -> rotation, append -> attention with the heads' scores mixed before the softmax
-//                  (mixed_head_attn.cu; temperature and scale folded into the mixing matrix) -> W_o.
+//                  (mixed_head_attn.cu) -> W_o.
 //   residual:      one kernel adds a sublayer's result (for experts: the weighted sum of a token's choices, in their order)
 //                  and writes the next sublayer's normed input.
 //   dense ff:      [W_gate; W_up] with rows interleaved and relu(gate) * up as the epilogue, then W_down.
@@ -43,7 +43,7 @@ struct KLayer {
     void *uk_t = nullptr, *uv = nullptr;         // (heads, rank_cols, dim), (heads * vdim, rank_cols)
     // differential / mixed heads
     float lambda = 0.f;
-    float* mix = nullptr;                        // (heads, heads), temperature and scale folded in
+    float *mix = nullptr, *factor = nullptr;     // (heads, heads), (heads): temperature times scale
     int rot = -1;                                // index into the model's rotation tables
     // feed-forward
     void* w_gu = nullptr;                        // dense (2 * ff, width), experts (experts, 2 * ff, width): rows 2j / 2j+1 = gate_j / up_j
@@ -250,11 +250,12 @@ int finalize_layer(zl_dekalorn* m, int l) {
         std::vector<double> temp, talk;
         RCHECK(take_host(m, mx + "temp", 1, H, temp));
         RCHECK(take_host(m, mx + "talk", H, H, talk));
-        std::vector<float> mix((size_t)H * H);
-        for (int h = 0; h < H; ++h)
-            for (int g = 0; g < H; ++g) mix[(size_t)h * H + g] = (float)(talk[(size_t)h * H + g] * temp[g] * (double)lc.scale);
+        std::vector<float> mix(talk.begin(), talk.end()), factor(H);
+        for (int h = 0; h < H; ++h) factor[h] = (float)(temp[h] * (double)lc.scale);
         RCHECK(dmalloc((void**)&L.mix, mix.size() * 4));
         ZL_CHECK_CUDA(cudaMemcpy(L.mix, mix.data(), mix.size() * 4, cudaMemcpyHostToDevice));
+        RCHECK(dmalloc((void**)&L.factor, factor.size() * 4));
+        ZL_CHECK_CUDA(cudaMemcpy(L.factor, factor.data(), factor.size() * 4, cudaMemcpyHostToDevice));
     }
     RCHECK(take_weight(m, mx + "o", D, H * vd, &L.o));
     if (lc.ff_kind != ZL_FF_NONE) RCHECK(finalize_ff(m, l));
@@ -269,11 +270,11 @@ int len_bucket(const zl_dekalorn* m, int max_len) {
     return b < m->cfg.max_seq ? b : (m->cfg.max_seq > 256 ? m->cfg.max_seq : 256);
 }
 
-int attn_splits(const zl_dekalorn_layer_t& lc, int rank_cols, int T, int max_len) {
+int attn_splits(const zl_dekalorn_layer_t& lc, int rank_cols, int T, int n_runs, int max_len) {
     const int len = lc.window > 0 && lc.window < max_len ? lc.window : max_len;
     if (lc.type == ZL_DEKALORN_LATENT) return zl_latent_attention_splits(T, lc.heads, rank_cols, max_len);
     if (lc.type == ZL_DEKALORN_DIFF) return zl_sink_attention_splits(T, lc.heads, lc.kv_heads, len);
-    return zl_mixed_head_attention_splits(T, lc.heads, len);
+    return zl_mixed_head_attention_splits(T, n_runs, lc.heads, lc.kv_heads, lc.dim, lc.vdim, len);
 }
 
 int alloc_runtime(zl_dekalorn* m) {
@@ -285,11 +286,12 @@ int alloc_runtime(zl_dekalorn* m) {
         const bool latent = lc.type == ZL_DEKALORN_LATENT;
         const int maps = lc.type == ZL_DEKALORN_DIFF ? 2 : 1;
         if (latent) RCHECK(zl_latent_attention_prepare_ex(lc.heads, L.rank_cols, L.row_cols, c.dtype));
+        // the split count falls as the rows grow and depends on how they form runs: size for the worst product
+        const int len = len_bucket(m, c.max_seq);
         for (int b = 1; b <= T; ++b) {
-            const int s = attn_splits(lc, L.rank_cols, b, len_bucket(m, c.max_seq));
+            const int s = std::max(attn_splits(lc, L.rank_cols, b, 1, len), attn_splits(lc, L.rank_cols, b, b, len));
             m->attn_ws_bytes = std::max(m->attn_ws_bytes, latent ? zl_latent_attention_workspace_bytes(b, lc.heads, L.rank_cols, s)
                                                                  : zl_sink_attention_workspace_bytes(b, lc.heads * maps, lc.vdim, s));
-            if (s == 1) break;
         }
         n_in = std::max(n_in, (size_t)L.n_in);
         hd = std::max(hd, (size_t)lc.heads * lc.dim * maps);
@@ -383,7 +385,7 @@ int enqueue_mixer(zl_dekalorn* m, KRun& U, int T, int n_runs, int max_run, int m
     const int pg = pdl_for(m, 2, T), pr = pdl_for(m, 4, T), pa = pdl_for(m, 8, T);
     cudaStream_t st = m->stream;
     const float* tab = L.rot >= 0 ? m->rots[L.rot].table : nullptr;
-    const int splits = attn_splits(lc, L.rank_cols, T, max_len);
+    const int splits = attn_splits(lc, L.rank_cols, T, n_runs, max_len);
     RCHECK(linear(m, m->h, D, L.w_in, L.n_in, m->proj, T, ZL_F32));
     if (lc.type == ZL_DEKALORN_LATENT) {
         const int RC = L.rank_cols, RS = L.row_cols;
@@ -406,7 +408,7 @@ int enqueue_mixer(zl_dekalorn* m, KRun& U, int T, int n_runs, int max_run, int m
     } else {
         RCHECK(zl_qkv_table_rope_append(m->proj, L.n_in, 0, L.k_off, L.v_off, H, G, d, vd, tab, lc.rot_dims, nullptr, ZL_ROT_ADJACENT,
                                         m->q, U.a.addrs, U.b.addrs, m->d_slots, m->d_pos, T, dt, pr, st));
-        RCHECK(zl_mixed_head_attention(m->q, U.a.addrs, U.b.addrs, m->d_slots, m->d_pos, L.mix, lc.window, m->att, T, H, G, d, vd,
+        RCHECK(zl_mixed_head_attention(m->q, U.a.addrs, U.b.addrs, m->d_slots, m->d_pos, L.mix, L.factor, lc.window, m->att, T, H, G, d, vd,
                                        splits, m->attn_ws, m->attn_ws_bytes, m->d_run0, m->d_runlen, n_runs, max_run, dt, pa, st));
     }
     return linear(m, m->att, H * vd, L.o, D, m->y, T, ZL_F32);
@@ -554,7 +556,7 @@ extern "C" void zl_dekalorn_destroy(zl_dekalorn_t* m) {
     for (auto& g : m->graphs) cudaGraphExecDestroy(g.second);
     for (auto& s : m->staged) cudaFree(s.second.ptr);
     for (auto& L : m->layers)
-        for (void* p : {(void*)L.norm1, (void*)L.norm2, L.w_in, L.o, (void*)L.dkv_norm, L.uk_t, L.uv, (void*)L.mix, L.w_gu, L.w_down,
+        for (void* p : {(void*)L.norm1, (void*)L.norm2, L.w_in, L.o, (void*)L.dkv_norm, L.uk_t, L.uv, (void*)L.mix, (void*)L.factor, L.w_gu, L.w_down,
                         L.router})
             if (p) cudaFree(p);
     for (auto& U : m->runs) {

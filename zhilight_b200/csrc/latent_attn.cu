@@ -764,12 +764,11 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
         }
         return;
     }
-    float keep[16], wv[16], ss = 0.f;   // the first 512 columns in registers, every load in flight at once
+    float keep[16], ss = 0.f;   // the first 512 columns in registers, every load in flight at once
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
         const int c = lane + 32 * i;
         keep[i] = c < p.R ? src[c] : 0.f;
-        wv[i] = c < p.R ? p.kv_w[c] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < 16; ++i) ss = fmaf(keep[i], keep[i], ss);
@@ -778,7 +777,7 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
         const int c = lane + 32 * i;
-        if (c < p.R) dst[c] = from_f32<TO>(keep[i] * r * wv[i]);
+        if (c < p.R) dst[c] = from_f32<TO>(keep[i] * r * p.kv_w[c]);
     }
     for (int c = lane + 512; c < p.R; c += 32) dst[c] = from_f32<TO>(src[c] * r * p.kv_w[c]);
 }

@@ -624,9 +624,10 @@ static cudaError_t launch_sink_mma_t(const SinkAttnMmaP& pp, int runs, int max_r
     return launch_sink_mma_d<T, 16, MAPS>(pp, runs, max_run_len, pdl, st);
 }
 
-// merge of the splits (at most 32) with the sink term and the gate; one warp per (token, head), grid (ceil(H / 4), T).
+// merge of the splits (at most MS: 4, 8 or 32) with the sink term and the gate; one warp per (token, head), grid
+// (ceil(H / 4), T).
 // Lane s holds the (max, sum) of split s, so the weights of all splits come from one round of loads.
-template <typename T>
+template <typename T, int MS>
 __global__ void __launch_bounds__(128) k_sink_attn_merge(SinkAttnP p) {
     pdl_trigger();
     pdl_wait();
@@ -645,41 +646,41 @@ __global__ void __launch_bounds__(128) k_sink_attn_merge(SinkAttnP p) {
     float gate = 1.0f;
     if (p.gate) gate = 1.0f / (1.0f + expf(-p.gate[(size_t)t * p.ldg + h]));
     T* out = static_cast<T*>(p.out) + ((size_t)t * p.H + h) * p.vd;
-    float wv[32];   // every split's weight in every lane: the loads below do not wait for shuffles
+    float wv[MS];   // every split's weight in every lane: the loads below do not wait for shuffles
 #pragma unroll
-    for (int s = 0; s < 32; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
+    for (int s = 0; s < MS; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
     if (p.out_table) {
         const float2* tab = reinterpret_cast<const float2*>(p.out_table) + (size_t)t * (p.vd >> 1);
         for (int mi = lane; mi < (p.vd >> 1); mi += 32) {
             int c1, c2;
             sa_pair(p, mi, c1, c2);
-            float v1[32], v2[32];
+            float v1[MS], v2[MS];
 #pragma unroll
-            for (int s = 0; s < 32; ++s) {
+            for (int s = 0; s < MS; ++s) {
                 v1[s] = s < p.splits ? part[(size_t)s * stride + 2 + c1] : 0.f;
                 v2[s] = s < p.splits ? part[(size_t)s * stride + 2 + c2] : 0.f;
             }
             float o1 = 0.f, o2 = 0.f;
 #pragma unroll
-            for (int s = 0; s < 32; ++s) o1 = fmaf(v1[s], wv[s], o1), o2 = fmaf(v2[s], wv[s], o2);
+            for (int s = 0; s < MS; ++s) o1 = fmaf(v1[s], wv[s], o1), o2 = fmaf(v2[s], wv[s], o2);
             sa_store_unrotated<T>(out, c1, c2, o1, o2, tab[mi], gate / L);
         }
         return;
     }
     for (int c = lane; c < p.vd; c += 32) {
-        float v[32];
+        float v[MS];
 #pragma unroll
-        for (int s = 0; s < 32; ++s) v[s] = s < p.splits ? part[(size_t)s * stride + 2 + c] : 0.f;   // all loads in flight
+        for (int s = 0; s < MS; ++s) v[s] = s < p.splits ? part[(size_t)s * stride + 2 + c] : 0.f;   // all loads in flight
         float o = 0.f;
 #pragma unroll
-        for (int s = 0; s < 32; ++s) o = fmaf(v[s], wv[s], o);   // splits in order; absent ones add 0 * 0
+        for (int s = 0; s < MS; ++s) o = fmaf(v[s], wv[s], o);   // splits in order; absent ones add 0 * 0
         out[c] = from_f32<T>(o / L * gate);
     }
 }
 
 // The same for two maps per head: a warp per map (two heads per CTA); the second map's merged sum goes through shared
 // memory to the first one's warp, which takes the difference, the norm over the head and the gate.
-template <typename T>
+template <typename T, int MS>
 __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
     __shared__ float second[2][32 * kSaMaxPerLane];
     pdl_trigger();
@@ -694,9 +695,9 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
         const float ls = lane < p.splits ? part[(size_t)lane * stride + 1] : 0.f;
         const float M = warp_max(ms);
         const float wgt = ms == -INFINITY ? 0.f : expf(ms - M);
-        float L = 0.f, wv[32];
+        float L = 0.f, wv[MS];
 #pragma unroll
-        for (int s = 0; s < 32; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
+        for (int s = 0; s < MS; ++s) wv[s] = __shfl_sync(0xffffffffu, wgt, s);
         for (int s = 0; s < p.splits; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, wgt, s), L);
         const float f = (map ? p.lambda : 1.0f) / L;
 #pragma unroll
@@ -704,12 +705,12 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
             const int c = lane + 32 * i;
             keep[i] = 0.f;
             if (c >= p.vd) continue;
-            float v[32];
+            float v[MS];
 #pragma unroll
-            for (int s = 0; s < 32; ++s) v[s] = s < p.splits ? part[(size_t)s * stride + 2 + c] : 0.f;   // all loads in flight
+            for (int s = 0; s < MS; ++s) v[s] = s < p.splits ? part[(size_t)s * stride + 2 + c] : 0.f;   // all loads in flight
             float o = 0.f;
 #pragma unroll
-            for (int s = 0; s < 32; ++s) o = fmaf(v[s], wv[s], o);
+            for (int s = 0; s < MS; ++s) o = fmaf(v[s], wv[s], o);
             keep[i] = o * f;
             if (map) second[w >> 1][c] = keep[i];
         }
@@ -735,10 +736,16 @@ __global__ void __launch_bounds__(128) k_two_map_merge(SinkAttnP p) {
     }
 }
 
+template <typename T, int MS>
+static cudaError_t sa_merge_ms(const SinkAttnP& p, int maps, int T_, bool pdl, cudaStream_t st) {
+    const dim3 mg(cdiv(p.H, maps == 2 ? 2 : 4), T_), mb(128);
+    return maps == 2 ? launch(k_two_map_merge<T, MS>, mg, mb, 0, st, pdl, p) : launch(k_sink_attn_merge<T, MS>, mg, mb, 0, st, pdl, p);
+}
 template <typename T>
 static cudaError_t sa_merge_t(const SinkAttnP& p, int maps, int T_, bool pdl, cudaStream_t st) {
-    const dim3 mg(cdiv(p.H, maps == 2 ? 2 : 4), T_), mb(128);
-    return maps == 2 ? launch(k_two_map_merge<T>, mg, mb, 0, st, pdl, p) : launch(k_sink_attn_merge<T>, mg, mb, 0, st, pdl, p);
+    if (p.splits <= 4) return sa_merge_ms<T, 4>(p, maps, T_, pdl, st);
+    if (p.splits <= 8) return sa_merge_ms<T, 8>(p, maps, T_, pdl, st);
+    return sa_merge_ms<T, 32>(p, maps, T_, pdl, st);
 }
 int sink_attn_merge(const SinkAttnP& p, int maps, int T, int dtype, bool pdl, cudaStream_t st) {
     cudaError_t e;

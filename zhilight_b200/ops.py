@@ -875,14 +875,14 @@ def window_attention(q, k_table, v_table, slot, pos, scale, window, heads, kv_he
     return out
 
 
-def mixed_head_attention(q, k_table, v_table, slot, pos, mix, window, heads, kv_heads, dim, vdim, splits=1, run_row0=None,
+def mixed_head_attention(q, k_table, v_table, slot, pos, mix, factor, window, heads, kv_heads, dim, vdim, splits=1, run_row0=None,
                          run_len=None, max_run_len=0):
-    """Attention whose heads' scores are mixed by mix (heads, heads) fp32 (the scale folded in) before the softmax."""
+    """Attention whose heads' scores, times factor (heads) fp32, are mixed by mix (heads, heads) fp32 before the softmax."""
     t = q.shape[0]
     nbytes = _lib.load().zl_sink_attention_workspace_bytes(t, heads, vdim, splits)
     ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=q.device)
     out = torch.empty((t, heads * vdim), dtype=q.dtype, device=q.device)
-    _lib.call("zl_mixed_head_attention", _p(q), _p(k_table), _p(v_table), _p(slot), _p(pos), _p(mix), window, _p(out), t, heads,
+    _lib.call("zl_mixed_head_attention", _p(q), _p(k_table), _p(v_table), _p(slot), _p(pos), _p(mix), _p(factor), window, _p(out), t, heads,
               kv_heads, dim, vdim, splits, _p(ws), nbytes, _p(run_row0), _p(run_len),
               run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(q), 0, _stream())
     return out
