@@ -743,11 +743,11 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
         const float* src = row + p.q_off + (size_t)unit * (p.d + p.rd);
         TO* dst = static_cast<TO*>(p.q_out) + ((size_t)t * p.H + unit) * p.d;
 #pragma unroll 4
-        for (int c = lane; c < p.d; c += 32) dst[c] = from_f32<TO>(src[c]);
+        for (int c = lane; c < p.d; c += 32) dst[c] = from_f32<TO>(__ldg(src + c));
         float* qr = p.qa + ((size_t)t * p.H + unit) * p.row_cols + p.rank_cols;
         for (int i = lane; i < (p.rd >> 1); i += 32) {
-            const float u = src[p.d + 2 * i], v = src[p.d + 2 * i + 1];
-            const float2 cs = tab[i];
+            const float u = __ldg(src + p.d + 2 * i), v = __ldg(src + p.d + 2 * i + 1);
+            const float2 cs = __ldg(tab + i);
             qr[2 * i] = u * cs.x - v * cs.y;
             qr[2 * i + 1] = v * cs.x + u * cs.y;
         }
@@ -768,7 +768,7 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
         const int c = lane + 32 * i;
-        keep[i] = c < p.R ? src[c] : 0.f;
+        keep[i] = c < p.R ? __ldg(src + c) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < 16; ++i) ss = fmaf(keep[i], keep[i], ss);
@@ -777,7 +777,7 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
         const int c = lane + 32 * i;
-        if (c < p.R) dst[c] = from_f32<TO>(keep[i] * r * p.kv_w[c]);
+        if (c < p.R) dst[c] = from_f32<TO>(keep[i] * r * __ldg(p.kv_w + c));
     }
     for (int c = lane + 512; c < p.R; c += 32) dst[c] = from_f32<TO>(src[c] * r * p.kv_w[c]);
 }
