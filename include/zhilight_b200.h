@@ -764,6 +764,66 @@ int zl_latent_attention_ex(const float* q_absorbed, void* const* slot_addrs, con
                            int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
                            const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
                            zl_stream_t stream);
+/* zl_rope_table with cos and sin times `mult` (in double before the rounding). */
+int zl_rope_table_scaled(const int32_t* pos, int T, const double* inv_freq, int half, double mult, float* table, int pdl,
+                         zl_stream_t stream);
+/* zl_qkv_headnorm_rope_append with values stored as projected (value_norm 0) and / or a query temperature: normed queries
+ * times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1) (temp_coef 0: none). */
+int zl_qkv_headnorm_append_ex(const float* proj, long long ldp, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim,
+                              int vdim, const float* q_weight, const float* k_weight, int value_norm, float temp_coef,
+                              double temp_every, const double* inv_freq, int rot_dims, float mscale, float eps, void* q_out,
+                              void* const* k_addrs, void* const* v_addrs, const int32_t* slot, const int32_t* pos, int T,
+                              int dtype, int pdl, zl_stream_t stream);
+/* zl_sink_attention_ex without gate, chunks and output rotation, with s = scale (q . k), then softcap tanh(s / softcap)
+ * (softcap 0: none), then minus slopes[head] * (pos - key) (slopes fp32 (heads) or NULL), and a sliding window (0: none).  The
+ * sink enters the denominator as it is. */
+int zl_biased_sink_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot, const int32_t* pos,
+                             const float* sink, int no_sink, float scale, float softcap, const float* slopes, int window, void* out,
+                             int T, int heads, int kv_heads, int dim, int vdim, int splits, void* workspace,
+                             size_t workspace_bytes, const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len,
+                             int dtype, int pdl, zl_stream_t stream);
+/* zl_latent_rope_append with the queries in a matrix of their own: query heads from q_proj (row stride ldq, head h at column
+ * h * (dim + rot_dim)), latent and rotated key part from kv_proj (row stride ldkv) at column c_off. */
+int zl_latent_rope_append_split(const float* q_proj, long long ldq, int heads, int dim, int rot_dim, const float* table, void* q_out,
+                                float* qa, const float* kv_proj, long long ldkv, int c_off, int kv_rank, const float* kv_weight,
+                                int rank_cols, int row_cols, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                                int T, float eps, int dtype, int pdl, zl_stream_t stream);
+/* zl_latent_attention_ex in a sliding window: token t sees the rows j with 0 <= pos[t] - j < window (0: all j <= pos[t]).
+ * Splits of zl_latent_attention_splits with max_len at most the window. */
+int zl_latent_window_attention(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                               const float* sink, const float* gate, long long ldg, float scale, int window, void* out, int T,
+                               int heads, int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
+                               const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
+                               zl_stream_t stream);
+/* Hyper-connections: the residual is `streams` fp32 copies per token, x (T, streams, D).  zl_hyper_update takes a sublayer's
+ * result y = sum_p coef[t][p] parts[t * n_parts + p] (coef NULL: ones) + dense[t] (NULL: none) into all streams at once,
+ * x_s' <- sum_s mix[s * streams + s'] x_s + out[s'] y, and reads the next sublayer's input u = sum_s in[s] x_s (in NULL: the sum
+ * of the streams): u to u_out (T, D) fp32 when not NULL, next_w * u / sqrt(mean(u^2) + eps) to h (T, D) of act_dtype when next_w
+ * is not NULL.  zl_hyper_embed starts the streams: x_s[t] = scale * table[ids[t]], with the same read. */
+int zl_hyper_update(float* x, int streams, const float* parts, long long ldp, const float* coef, int n_parts, const float* dense,
+                    long long ldd, const float* mix, const float* out, const float* in, const float* next_w, void* h,
+                    float* u_out, int act_dtype, int T, int D, float eps, int pdl, zl_stream_t stream);
+int zl_hyper_embed(const int32_t* ids, const void* table, int vocab, float scale, float* x, int streams, const float* in,
+                   const float* next_w, void* h, float* u_out, int act_dtype, int T, int D, float eps, int pdl,
+                   zl_stream_t stream);
+/* Selective state space (state-space duality form): head h of `heads` keeps S (state x vdim) and reads the B and C vectors of
+ * group h / (heads / groups).  proj (T, ld) fp32 holds x | B | C (heads * vdim, groups * state, groups * state channels) at
+ * column col_x and one step-size logit per head at col_dt.  x, B and C pass a causal convolution per channel over the
+ * sequence's positions (conv_weight (taps, channels) fp32, the last tap is the current token's, conv_bias (channels), zeros
+ * before the start) and silu; dt = softplus(logit + dt_bias[h]);
+ *   S_t = exp(-exp(a_log[h]) dt) S_(t-1) + dt B_t x_t^T,   o_t = S_t^T C_t + d_skip[h] x_t.
+ * ring_addrs: slot -> (taps - 1, channels) fp32 (the input at position p in entry p % (taps - 1)); state_addrs: slot ->
+ * (heads, vdim, state) fp32; a run that starts at position 0 starts from zero.  o (T, heads * vdim) fp32.  Everything is fp32. */
+size_t zl_ssm_workspace_bytes(int T, int heads, int vdim, int state, int groups);
+int zl_ssm_prepare(int vdim, int state);
+int zl_ssm_scan(const float* proj, long long ld, int col_x, int col_dt, const float* conv_weight, const float* conv_bias, int taps,
+                const float* dt_bias, const float* a_log, const float* d_skip, void* const* ring_addrs, const int32_t* run_row0,
+                const int32_t* run_len, int runs, const int32_t* slot, const int32_t* pos, void* const* state_addrs, float* o,
+                long long ld_o, int heads, int vdim, int state, int groups, int T, void* workspace, size_t workspace_bytes, int pdl,
+                zl_stream_t stream);
+/* y[t] (of out_dtype) = weight * v / sqrt(mean(v^2) + eps) in `groups` equal parts (each by its own mean), v = o[t] * silu(z[t]). */
+int zl_silu_gate_group_rmsnorm(const float* o, long long ldo, const float* z, long long ldz, const float* weight, void* y,
+                               long long ldy, int T, int D, int groups, float eps, int out_dtype, int pdl, zl_stream_t stream);
 /* ------------------------------------------------------------------------------------------ *
  * Kodupel: decoder-only model whose layers are listed one by one: the mixer is attention (grouped key/value heads,
  * biased projections, per-head query / key RMS norm, partial rotation in adjacent pairs with YaRN frequencies, value
@@ -957,6 +1017,56 @@ int zl_dekalorn_stats(zl_dekalorn_t* m, double* weight_bytes, int* kernels_per_s
  * and rotated key parts (n_rows, rot_dim); otherwise keys (n_rows, kv_heads * dim, twice that for differential attention)
  * and values (n_rows, kv_heads * vdim). */
 int zl_dekalorn_read_cache(zl_dekalorn_t* m, int run, int slot, int n_rows, float* a_host, float* b_host);
+/* ------------------------------------------------------------------------------------------ *
+ * Bezasun: decoder-only model of pre-norm layers (RMS norm with weight 1 + w), listed one by one, on a residual of `streams`
+ * fp32 copies joined by hyper-connections (zl_hyper_update).  The mixer is grouped-query attention without positions (per-head
+ * query / key norms, query temperature, soft-capped scores with a linear distance bias, a sink per head), latent attention in
+ * a sliding window (queries through a normed latent, one rotated key part with YaRN frequencies shared by the heads), or a
+ * selective state space behind a short convolution with a silu gate and a norm in groups.  The feed-forward is absent or
+ * a mixture of silu-gated experts weighted by their softmax scores, plus an optional shared expert.  Same driver shape as
+ * zl_dekalorn_*.
+ * ------------------------------------------------------------------------------------------ */
+enum { ZL_BEZASUN_ATTENTION = 0, ZL_BEZASUN_LATENT = 1, ZL_BEZASUN_SSM = 2 };
+typedef struct zl_bezasun zl_bezasun_t;
+typedef struct zl_bezasun_layer {
+    int type;                              /* ZL_BEZASUN_* */
+    int heads, kv_heads, dim, vdim;        /* kv_heads: attention; dim: head size (latent attention: unrotated part) */
+    float scale, softcap, temp_coef;       /* score scale; attention: 0 = no cap, 0 = no query temperature */
+    double temp_every;
+    int rot_dim, q_rank, kv_rank, window;  /* latent attention; window 0: none */
+    double rot_base, rot_factor /* 0: frequencies are not scaled */, rot_original, rot_fast, rot_slow;
+    int state, groups, conv, norm_groups;  /* state space: state size, groups of B / C, convolution taps, parts of the norm */
+    int ff_kind;                           /* ZL_FF_NONE or ZL_FF_MOE */
+    int ff, experts, top, shared_ff;       /* shared_ff 0: no shared expert */
+} zl_bezasun_layer_t;
+typedef struct zl_bezasun_config {
+    int num_layers, width, vocab, streams;
+    float eps, embed_scale, residual_mult, logit_scale;
+    int dtype; /* ZL_BF16 or ZL_F32 */
+    int max_batch, max_seq, max_step_tokens;
+    int use_pdl, use_graph;
+} zl_bezasun_config_t;
+int zl_bezasun_create(const zl_bezasun_config_t* cfg, const zl_bezasun_layer_t* layers, zl_bezasun_t** out);
+void zl_bezasun_destroy(zl_bezasun_t* m);
+int zl_bezasun_load_tensor(zl_bezasun_t* m, const char* name, const void* data_host, int rows, int cols, int elem_bytes);
+int zl_bezasun_init_synthetic(zl_bezasun_t* m, uint64_t seed);
+int zl_bezasun_finalize(zl_bezasun_t* m);
+/* As zl_dekipel_step. */
+int zl_bezasun_step(zl_bezasun_t* m, const int32_t* tokens_host, const int32_t* slots_host, const int32_t* positions_host,
+                    int T, const int32_t* want_rows_host, int n_want, float* logits_host, int32_t* next_host);
+int zl_bezasun_set_state(zl_bezasun_t* m, const int32_t* tokens_host, const int32_t* positions_host, int B);
+int zl_bezasun_step_device(zl_bezasun_t* m, int B);
+int zl_bezasun_sync(zl_bezasun_t* m);
+zl_stream_t zl_bezasun_stream(zl_bezasun_t* m);
+/* sum of the streams after every layer of the last step, (layers, T, width) fp32, when capture was switched on */
+int zl_bezasun_capture_layers(zl_bezasun_t* m, int on);
+int zl_bezasun_read_layers(zl_bezasun_t* m, float* out_host, int T);
+int zl_bezasun_stats(zl_bezasun_t* m, double* weight_bytes, int* kernels_per_step);
+/* Rows 0 .. n_rows of what layer `layer` caches for one slot, as fp32 (tests): latent attention: latents (n_rows, kv_rank) and
+ * rotated key parts (n_rows, rot_dim); attention: keys (n_rows, kv_heads * dim) and values (n_rows, kv_heads * vdim). */
+int zl_bezasun_read_cache(zl_bezasun_t* m, int layer, int slot, int n_rows, float* a_host, float* b_host);
+/* One slot's state of a state-space layer, (heads, vdim, state) fp32 (tests). */
+int zl_bezasun_read_state(zl_bezasun_t* m, int layer, int slot, float* out_host);
 #ifdef __cplusplus
 }
 #endif

@@ -96,6 +96,8 @@ def parse_header(path=HEADER):
     src = re.sub(r"typedef struct zl_dizizen_config \{.*?\} zl_dizizen_config_t;", " ", src, flags=re.S)
     src = re.sub(r"typedef struct zl_dekalorn_layer \{.*?\} zl_dekalorn_layer_t;", " ", src, flags=re.S)
     src = re.sub(r"typedef struct zl_dekalorn_config \{.*?\} zl_dekalorn_config_t;", " ", src, flags=re.S)
+    src = re.sub(r"typedef struct zl_bezasun_layer \{.*?\} zl_bezasun_layer_t;", " ", src, flags=re.S)
+    src = re.sub(r"typedef struct zl_bezasun_config \{.*?\} zl_bezasun_config_t;", " ", src, flags=re.S)
     src = re.sub(r"enum \{.*?\};", " ", src, flags=re.S)
     protos = {}
     for m in re.finditer(r"([A-Za-z_][\w \*]*?)\b(zl_\w+)\s*\(([^;{}]*?)\)\s*;", src):

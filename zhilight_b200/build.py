@@ -37,6 +37,8 @@ FAMILY_SOURCES = {
     "lagelorn": _FP32_RESIDUAL_COMMON + ["mixer_rows", "delta_rule", "sink_attn", "lagelorn_runner"],
     "dekalorn": _FP32_RESIDUAL_COMMON + ["mixer_rows", "moe_route", "sink_attn", "latent_attn", "mixed_head_attn",
                                          "dekalorn_runner"],
+    "bezasun": _FP32_RESIDUAL_COMMON + ["mixer_rows", "moe_route", "sink_attn", "latent_attn", "hyper_residual", "ssm_scan",
+                                        "bezasun_runner"],
     "dizizen": _FP32_RESIDUAL_COMMON + ["mixer_rows", "moe_route", "sink_attn", "dizizen_runner"],
 }
 

@@ -15,7 +15,8 @@
 // General form (zl_latent_attention_ex): a cached row may carry more columns than the value has -- a rotated key part
 // shared by the heads behind the latent -- that enter the score only; the sink may be absent (an ordinary softmax); a
 // sigmoid gate per head may multiply the output; and the probabilities may enter the 16-bit product as a hi + lo pair,
-// so that no weight is rounded to 8 bits.  k_latent_rope_append writes such rows and the queries' rotated parts.
+// so that no weight is rounded to 8 bits; and a sliding window may restrict a token to the last `window` rows up to its own.
+// k_latent_rope_append writes such rows and the queries' rotated parts.
 #include "common.cuh"
 
 #include <math.h>
@@ -42,7 +43,14 @@ struct LaParams {
     int RS;                // columns of a cached row and of qa: the score runs over all of them, the value is the first R
     const float* gate = nullptr;   // gate[t * ldg + h] logits or null
     long long ldg = 0;
+    int window = 0;                // > 0: rows at distance >= window are not seen
 };
+
+// first row a token at `pos` sees
+template <typename TC>
+__device__ __forceinline__ int la_first_row(const LaParams<TC>& p, int pos) {
+    return p.window > 0 && pos >= p.window ? pos - p.window + 1 : 0;
+}
 
 __device__ __forceinline__ float la_gate(const float* gate, long long ldg, int t, int h) {
     return gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h])) : 1.0f;
@@ -65,10 +73,10 @@ __global__ void __launch_bounds__(kLaThreads) k_latent_attn(LaParams<TC> p) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int len = p.pos[t] + 1;
     const TC* cache = static_cast<const TC*>(p.slot_addrs[p.slot[t]]);
-    int lo = 0, hi = len;
+    int lo = la_first_row(p, len - 1), hi = len;
     if (p.S > 1) {
-        const int per = cdiv(cdiv(len, p.S), kLaKeys) * kLaKeys;
-        lo = split * per;
+        const int per = cdiv(cdiv(len - lo, p.S), kLaKeys) * kLaKeys;
+        lo += split * per;
         hi = min(len, lo + per);
     }
     for (int i = tid; i < hg * RS; i += kLaThreads) sq[i] = p.qa[((size_t)t * p.H + h0) * RS + i];
@@ -220,10 +228,10 @@ __global__ void __launch_bounds__(128) k_latent_attn_mma(LaParams<__nv_bfloat16>
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
     const int len = p.pos[t] + 1;
     const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.slot_addrs[p.slot[t]]);
-    int lo = 0, hi = len;
+    int lo = la_first_row(p, len - 1), hi = len;
     if (p.S > 1) {
-        const int per = cdiv(cdiv(len, p.S), kLmKeys) * kLmKeys;
-        lo = split * per;
+        const int per = cdiv(cdiv(len - lo, p.S), kLmKeys) * kLmKeys;
+        lo += split * per;
         hi = min(len, lo + per);
     }
     const int ha = h0 + g, hb = h0 + g + 8;   // the two heads (rows) this lane holds
@@ -435,10 +443,11 @@ __global__ void __launch_bounds__(256, 1) k_latent_tile_mma(LaTileP pp) {
     const int ntok = min(pp.nq, len - t0), row0 = pp.run_row0[run] + t0, hb = pp.hb, hn = min(hb, H - h0);
     const int pos0 = p.pos[row0];
     const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.slot_addrs[p.slot[row0]]);
-    int lo = 0, hi = pos0 + ntok;
+    // row tiles start at multiples of kLtKeys from row 0 whatever the step, so a token's sums do not depend on the cut
+    int lo = la_first_row(p, pos0) / kLtKeys * kLtKeys, hi = pos0 + ntok;
     if (p.S > 1) {
-        const int per = cdiv(cdiv(hi, p.S), kLtKeys) * kLtKeys;
-        lo = split * per;
+        const int per = cdiv(cdiv(hi - lo, p.S), kLtKeys) * kLtKeys;
+        lo += split * per;
         hi = min(hi, lo + per);
     }
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
@@ -453,7 +462,7 @@ __global__ void __launch_bounds__(256, 1) k_latent_tile_mma(LaTileP pp) {
             }
         cp_async_commit();
     };
-    int t_of[2], h_of[2], pos_of[2];
+    int t_of[2], h_of[2], pos_of[2], first_of[2];
     bool ok[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -462,6 +471,7 @@ __global__ void __launch_bounds__(256, 1) k_latent_tile_mma(LaTileP pp) {
         h_of[i] = h0 + r - tk * hb;
         ok[i] = tk < ntok && h_of[i] < H;
         pos_of[i] = ok[i] ? pos0 + tk : -1;
+        first_of[i] = la_first_row(p, pos_of[i]);
     }
     float m_run[2], l_run[2];
 #pragma unroll
@@ -530,8 +540,8 @@ __global__ void __launch_bounds__(256, 1) k_latent_tile_mma(LaTileP pp) {
             for (int i = 0; i < 2; ++i) {
                 const float2 x = *reinterpret_cast<const float2*>(sr + (size_t)(g + i * 8) * kLtSp + nt * 8 + 2 * q4);
                 const int j = j0 + nt * 8 + 2 * q4;
-                v[nt][2 * i] = j < hi && j <= pos_of[i] ? x.x * p.scale : -INFINITY;
-                v[nt][2 * i + 1] = j + 1 < hi && j + 1 <= pos_of[i] ? x.y * p.scale : -INFINITY;
+                v[nt][2 * i] = j < hi && j <= pos_of[i] && j >= first_of[i] ? x.x * p.scale : -INFINITY;
+                v[nt][2 * i + 1] = j + 1 < hi && j + 1 <= pos_of[i] && j + 1 >= first_of[i] ? x.y * p.scale : -INFINITY;
                 mx[i] = fmaxf(mx[i], fmaxf(v[nt][2 * i], v[nt][2 * i + 1]));
             }
         float corr[2], sum[2] = {0.f, 0.f};
@@ -718,8 +728,10 @@ static int la_launch(LaParams<TC> p, int T, bool pdl, cudaStream_t st) {
 
 // one warp per (token, unit): the H query heads, then the rotated key part, then the latent (norm and append)
 struct LaPrepP {
-    const float* proj;
+    const float* proj;         // the queries' matrix
     long long ldp;
+    const float* kv;           // the latents' matrix (the same one, or its own)
+    long long ldkv;
     int q_off, H, d, rd;
     const float2* table;       // (T, rd / 2)
     void* q_out;
@@ -754,7 +766,7 @@ __global__ void __launch_bounds__(256) k_latent_rope_append(LaPrepP p) {
         return;
     }
     TO* dst = static_cast<TO*>(p.slot_addrs[p.slot[t]]) + (size_t)p.pos[t] * p.row_cols;
-    const float* src = row + p.c_off;
+    const float* src = p.kv + (size_t)t * p.ldkv + p.c_off;
     if (unit == p.H) {
         for (int i = lane; i < (p.rd >> 1); i += 32) {
             const float u = src[p.R + 2 * i], v = src[p.R + 2 * i + 1];
@@ -836,11 +848,11 @@ extern "C" int zl_latent_attention_prepare_ex(int heads, int rank_cols, int row_
 template <typename TC>
 static LaParams<TC> la_params(const float* qa, void* const* slot_addrs, const int32_t* slot, const int32_t* pos, const float* sink,
                               float scale, void* out, int T, int heads, int R, int RS, int splits, void* workspace,
-                              const float* gate, long long ldg) {
+                              const float* gate, long long ldg, int window = 0) {
     float* part_acc = static_cast<float*>(workspace);
     float* part_ml = splits > 1 ? part_acc + (size_t)T * heads * splits * R : nullptr;
     return LaParams<TC>{qa, slot_addrs, slot, pos, sink, out, part_acc, part_ml, scale, heads, R, la_heads_per_cta(heads, R), splits,
-                        RS, gate, ldg};
+                        RS, gate, ldg, window};
 }
 
 extern "C" int zl_latent_attention(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
@@ -862,6 +874,16 @@ extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot
                                       int heads, int rank_cols, int row_cols, int splits, void* workspace, size_t workspace_bytes,
                                       const int32_t* run_row0, const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl,
                                       zl_stream_t stream) {
+    return zl_latent_window_attention(q_absorbed, slot_addrs, slot, pos, sink, gate, ldg, scale, 0, out, T, heads, rank_cols, row_cols,
+                                      splits, workspace, workspace_bytes, run_row0, run_len, runs, max_run_len, dtype, pdl, stream);
+}
+
+extern "C" int zl_latent_window_attention(const float* q_absorbed, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                                          const float* sink, const float* gate, long long ldg, float scale, int window, void* out,
+                                          int T, int heads, int rank_cols, int row_cols, int splits, void* workspace,
+                                          size_t workspace_bytes, const int32_t* run_row0, const int32_t* run_len, int runs,
+                                          int max_run_len, int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(window >= 0);
     ZL_CHECK_ARG(q_absorbed && slot_addrs && slot && pos && out && T > 0 && T <= 65535 && heads > 0 && rank_cols > 0);
     ZL_CHECK_ARG(row_cols >= rank_cols && (dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32));
     ZL_CHECK_ARG(splits >= 1 && splits <= 64 && heads <= 65535);
@@ -869,7 +891,7 @@ extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot
     ZL_CHECK_ARG(workspace_bytes >= zl_latent_attention_workspace_bytes(T, heads, rank_cols, splits) && (splits == 1 || workspace));
     ZL_CHECK_SUPPORTED(la_smem_bytes(la_heads_per_cta(heads, rank_cols), row_cols) <= 200 * 1024);
 #define ZL_LA_P(TC) \
-    la_params<TC>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, rank_cols, row_cols, splits, workspace, gate, ldg)
+    la_params<TC>(q_absorbed, slot_addrs, slot, pos, sink, scale, out, T, heads, rank_cols, row_cols, splits, workspace, gate, ldg, window)
     if (dtype == ZL_F32) return la_launch<float>(ZL_LA_P(float), T, pdl != 0, stream);
     if (dtype == ZL_F16) return la_launch<__half>(ZL_LA_P(__half), T, pdl != 0, stream);
     const bool mma = lm_eligible_ex(dtype, rank_cols, row_cols) && row_cols % 8 == 0 && (reinterpret_cast<uintptr_t>(q_absorbed) & 15) == 0;
@@ -884,14 +906,14 @@ extern "C" int zl_latent_attention_ex(const float* q_absorbed, void* const* slot
 #undef ZL_LA_P
 }
 
-extern "C" int zl_latent_rope_append(const float* proj, long long ldp, int q_off, int heads, int dim, int rot_dim,
-                                     const float* table, void* q_out, float* qa, int c_off, int kv_rank, const float* kv_weight,
-                                     int rank_cols, int row_cols, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
-                                     int T, float eps, int dtype, int pdl, zl_stream_t stream) {
-    ZL_CHECK_ARG(proj && q_out && qa && kv_weight && slot_addrs && slot && pos && T > 0 && T <= 65535 && heads > 0 && dim > 0);
+static int latent_append(const float* q_proj, long long ldq, int q_off, int heads, int dim, int rot_dim, const float* table, void* q_out,
+                         float* qa, const float* kv_proj, long long ldkv, int c_off, int kv_rank, const float* kv_weight,
+                         int rank_cols, int row_cols, void* const* slot_addrs, const int32_t* slot, const int32_t* pos, int T,
+                         float eps, int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(q_proj && kv_proj && q_out && qa && kv_weight && slot_addrs && slot && pos && T > 0 && T <= 65535 && heads > 0 && dim > 0);
     ZL_CHECK_ARG(kv_rank > 0 && rank_cols >= kv_rank && rot_dim >= 0 && rot_dim % 2 == 0 && row_cols >= rank_cols + rot_dim);
     ZL_CHECK_ARG((rot_dim == 0 || table) && (dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32));
-    const LaPrepP p{proj, ldp, q_off, heads, dim, rot_dim, reinterpret_cast<const float2*>(table), q_out, qa, c_off, kv_rank, kv_weight,
+    const LaPrepP p{q_proj, ldq, kv_proj, ldkv, q_off, heads, dim, rot_dim, reinterpret_cast<const float2*>(table), q_out, qa, c_off, kv_rank, kv_weight,
                     rank_cols, row_cols, slot_addrs, slot, pos, eps};
     const dim3 grid(cdiv(heads + 2, 8), T), block(256);
     cudaError_t e;
@@ -900,4 +922,21 @@ extern "C" int zl_latent_rope_append(const float* proj, long long ldp, int q_off
     else e = launch(k_latent_rope_append<__half>, grid, block, 0, stream, pdl != 0, p);
     ZL_CHECK_CUDA(e);
     return ZL_OK;
+}
+
+extern "C" int zl_latent_rope_append(const float* proj, long long ldp, int q_off, int heads, int dim, int rot_dim,
+                                     const float* table, void* q_out, float* qa, int c_off, int kv_rank, const float* kv_weight,
+                                     int rank_cols, int row_cols, void* const* slot_addrs, const int32_t* slot, const int32_t* pos,
+                                     int T, float eps, int dtype, int pdl, zl_stream_t stream) {
+    return latent_append(proj, ldp, q_off, heads, dim, rot_dim, table, q_out, qa, proj, ldp, c_off, kv_rank, kv_weight, rank_cols,
+                         row_cols, slot_addrs, slot, pos, T, eps, dtype, pdl, stream);
+}
+
+extern "C" int zl_latent_rope_append_split(const float* q_proj, long long ldq, int heads, int dim, int rot_dim, const float* table,
+                                           void* q_out, float* qa, const float* kv_proj, long long ldkv, int c_off, int kv_rank,
+                                           const float* kv_weight, int rank_cols, int row_cols, void* const* slot_addrs,
+                                           const int32_t* slot, const int32_t* pos, int T, float eps, int dtype, int pdl,
+                                           zl_stream_t stream) {
+    return latent_append(q_proj, ldq, 0, heads, dim, rot_dim, table, q_out, qa, kv_proj, ldkv, c_off, kv_rank, kv_weight, rank_cols,
+                         row_cols, slot_addrs, slot, pos, T, eps, dtype, pdl, stream);
 }

@@ -1,7 +1,8 @@
 // Token-wise pieces of mixers that work per head, all in fp32 (rotation angles in double) with stores rounded to the
 // activation dtype:
 //   * the step from a fused q | k | v projection row to attention operands: RMS norm per head over the head size with a
-//     weight shared by the heads (queries, keys), a weightless RMS norm of every value head, a rotation of the first
+//     weight shared by the heads (queries, keys), an optional query temperature that grows with the logarithm of the position,
+//     an optional weightless RMS norm of every value head, a rotation of the first
 //     `rot_dims` dimensions of queries and keys in adjacent pairs (2i, 2i+1) by pos * inv_freq[i] with cos / sin scaled
 //     by `mscale` (the frequencies are a table, so any scaling rule is the caller's), and the append of keys and values
 //     to the slot's caches;
@@ -37,6 +38,9 @@ struct QkvPrepP {
     void* const* k_addrs;      // slot -> (max_seq, G, d)
     void* const* v_addrs;      // slot -> (max_seq, G, vd)
     const int32_t *slot, *pos;
+    int v_norm = 1;            // 0: values are stored as projected
+    float temp_coef = 0.f;     // normed queries times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1)
+    double temp_every = 1.0;
 };
 
 // one warp per (token, unit); units: H query heads, then G key heads, then G value heads.  grid (ceil(units / 4), T)
@@ -76,9 +80,14 @@ __global__ void __launch_bounds__(128) k_qkv_headnorm_rope_append(QkvPrepP p) {
         rotate = false;
         dst = static_cast<TO*>(p.v_addrs[p.slot[t]]) + ((size_t)pos * p.G + g) * p.vd;
     }
+    if (!w && !p.v_norm) {
+        for (int c = lane; c < n; c += 32) dst[c] = from_f32<TO>(src[c]);
+        return;
+    }
     float ss = 0.f;
     for (int c = lane; c < n; c += 32) ss = fmaf(src[c], src[c], ss);
-    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+    float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+    if (unit < p.H && p.temp_coef != 0.f) r *= 1.0f + p.temp_coef * logf((float)(floor((double)(pos + 1) / p.temp_every) + 1.0));
     const int rot = rotate ? p.rot_dims : 0;
     // rotated pairs: lane handles pair i = (2i, 2i + 1)
     for (int i = lane; 2 * i < rot; i += 32) {
@@ -348,10 +357,10 @@ __global__ void __launch_bounds__(256) k_postnorm_combine(float* __restrict__ x,
     }
 }
 
-// table[t][i] = (cos, sin)(pos[t] * inv_freq[i]): the angle and its functions in double (at position 1000 a float angle is
+// table[t][i] = (cos, sin)(pos[t] * inv_freq[i]) * mult: the angle and its functions in double (at position 1000 a float angle is
 // already off by 3e-5 rad), once per step for every kernel that turns by these angles
 __global__ void __launch_bounds__(256) k_rope_table(const int32_t* __restrict__ pos, const double* __restrict__ inv_freq,
-                                                    float2* __restrict__ table, int T, int half) {
+                                                    float2* __restrict__ table, int T, int half, double mult) {
     pdl_trigger();
     pdl_wait();
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -359,7 +368,7 @@ __global__ void __launch_bounds__(256) k_rope_table(const int32_t* __restrict__ 
     const int t = i / half;
     double sd, cd;
     sincos((double)pos[t] * inv_freq[i - t * half], &sd, &cd);
-    table[i] = make_float2((float)cd, (float)sd);
+    table[i] = make_float2((float)(cd * mult), (float)(sd * mult));
 }
 
 struct QkvRopeP {
@@ -732,9 +741,14 @@ extern "C" int zl_rope_inv_freq_wavelength(double base, int dims, double factor,
 
 extern "C" int zl_rope_table(const int32_t* pos, int T, const double* inv_freq, int half, float* table, int pdl,
                              zl_stream_t stream) {
+    return zl_rope_table_scaled(pos, T, inv_freq, half, 1.0, table, pdl, stream);
+}
+
+extern "C" int zl_rope_table_scaled(const int32_t* pos, int T, const double* inv_freq, int half, double mult, float* table, int pdl,
+                                    zl_stream_t stream) {
     ZL_CHECK_ARG(pos && inv_freq && table && T > 0 && half > 0 && (reinterpret_cast<uintptr_t>(table) & 7) == 0);
     ZL_CHECK_CUDA(launch(k_rope_table, dim3(cdiv(T * half, 256)), dim3(256), 0, stream, pdl != 0, pos, inv_freq,
-                         reinterpret_cast<float2*>(table), T, half));
+                         reinterpret_cast<float2*>(table), T, half, mult));
     return ZL_OK;
 }
 
@@ -888,12 +902,22 @@ extern "C" int zl_qkv_headnorm_rope_append(const float* proj, long long ldp, int
                                            const double* inv_freq, int rot_dims, float mscale, float eps, void* q_out,
                                            void* const* k_addrs, void* const* v_addrs, const int32_t* slot,
                                            const int32_t* pos, int T, int dtype, int pdl, zl_stream_t stream) {
+    return zl_qkv_headnorm_append_ex(proj, ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, q_weight, k_weight, 1, 0.f, 1.0,
+                                     inv_freq, rot_dims, mscale, eps, q_out, k_addrs, v_addrs, slot, pos, T, dtype, pdl, stream);
+}
+
+extern "C" int zl_qkv_headnorm_append_ex(const float* proj, long long ldp, int q_off, int k_off, int v_off, int heads,
+                                         int kv_heads, int dim, int vdim, const float* q_weight, const float* k_weight,
+                                         int value_norm, float temp_coef, double temp_every, const double* inv_freq, int rot_dims,
+                                         float mscale, float eps, void* q_out, void* const* k_addrs, void* const* v_addrs,
+                                         const int32_t* slot, const int32_t* pos, int T, int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(temp_coef == 0.f || temp_every > 0);
     ZL_CHECK_ARG(proj && q_weight && q_out && slot && pos && T > 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0);
     ZL_CHECK_ARG(rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq));
     ZL_CHECK_ARG(k_off < 0 || (k_weight && k_addrs && v_addrs && v_off >= 0));
     ZL_CHECK_ARG(dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32);
     QkvPrepP p{proj, ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, rot_dims, q_weight, k_weight, inv_freq,
-               mscale, eps, q_out, k_addrs, v_addrs, slot, pos};
+               mscale, eps, q_out, k_addrs, v_addrs, slot, pos, value_norm != 0, temp_coef, temp_every};
     const int units = heads + (k_off >= 0 ? 2 * kv_heads : 0);
     const dim3 grid(cdiv(units, 4), T), block(128);
     cudaError_t e;

@@ -297,4 +297,72 @@ int put_interleaved(M* m, const std::string& a, const std::string& b, int rows, 
     return ZL_OK;
 }
 
+// ---- load helpers of drivers with absorbed latent attention or small host-side tables --------------------------------------
+inline int round_up(int a, int b) { return (a + b - 1) / b * b; }
+
+// W_uk (H * d, R) -> (H, rank_cols, d): the per-head transpose, zero rows beyond R
+template <typename TS, typename TD>
+__global__ void k_uk_transpose(const TS* __restrict__ src, TD* __restrict__ dst, int H, int d, int R, int RC) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (size_t)H * RC * d) return;
+    const int c = (int)(i % d), r = (int)(i / d % RC), h = (int)(i / d / RC);
+    dst[i] = from_f32<TD>(r < R ? to_f32<TS>(src[((size_t)h * d + c) * R + r]) : 0.f);
+}
+// (rows, cols) -> (rows, cols_out), zero columns beyond cols
+template <typename TS, typename TD>
+__global__ void k_pad_cols(const TS* __restrict__ src, TD* __restrict__ dst, int rows, int cols, int cols_out) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (size_t)rows * cols_out) return;
+    const int c = (int)(i % cols_out);
+    dst[i] = from_f32<TD>(c < cols ? to_f32<TS>(src[i / cols_out * cols + c]) : 0.f);
+}
+
+template <typename TS, typename TD>
+void launch_uk_uv(bool uk, const void* src, void* dst, int H, int n, int R, int RC, cudaStream_t st) {
+    const unsigned blocks = (unsigned)(((size_t)H * RC * n + 255) / 256);
+    if (uk) k_uk_transpose<TS, TD><<<blocks, 256, 0, st>>>(static_cast<const TS*>(src), static_cast<TD*>(dst), H, n, R, RC);
+    else k_pad_cols<TS, TD><<<blocks, 256, 0, st>>>(static_cast<const TS*>(src), static_cast<TD*>(dst), H * n, R, RC);
+}
+
+// W_uk (transposed per head) or W_uv with its latent columns padded
+template <typename M>
+int take_latent(M* m, const std::string& name, bool uk, int H, int n, int R, int RC, void** out) {
+    const Staged* s = need(m, name, H * n, R);
+    if (!s) return ZL_ERR_STATE;
+    RCHECK(dmalloc(out, (size_t)H * n * RC * m->esz));
+    if (m->cfg.dtype == ZL_F32) {
+        if (s->elem == 2) launch_uk_uv<__nv_bfloat16, float>(uk, s->ptr, *out, H, n, R, RC, m->stream);
+        else launch_uk_uv<float, float>(uk, s->ptr, *out, H, n, R, RC, m->stream);
+    } else {
+        if (s->elem == 2) launch_uk_uv<__nv_bfloat16, __nv_bfloat16>(uk, s->ptr, *out, H, n, R, RC, m->stream);
+        else launch_uk_uv<float, __nv_bfloat16>(uk, s->ptr, *out, H, n, R, RC, m->stream);
+    }
+    ZL_CHECK_LAUNCH();
+    ZL_CHECK_CUDA(cudaStreamSynchronize(m->stream));
+    staged_drop(m->staged, name);
+    m->weight_bytes += (double)H * n * RC * m->esz;
+    return ZL_OK;
+}
+
+// a small staged tensor as doubles on the host
+template <typename M>
+int take_host(M* m, const std::string& name, int rows, int cols, std::vector<double>& out) {
+    float* d = nullptr;
+    RCHECK(take_f32(m, name, rows, cols, &d));
+    std::vector<float> f((size_t)rows * cols);
+    const cudaError_t e = cudaMemcpy(f.data(), d, f.size() * 4, cudaMemcpyDeviceToHost);
+    cudaFree(d);
+    ZL_CHECK_CUDA(e);
+    out.assign(f.begin(), f.end());
+    return ZL_OK;
+}
+
+// doubles computed on the host -> a new fp32 device array
+inline int upload_f32(const std::vector<double>& v, float** out) {
+    const std::vector<float> f(v.begin(), v.end());
+    RCHECK(dmalloc((void**)out, f.size() * 4));
+    ZL_CHECK_CUDA(cudaMemcpy(*out, f.data(), f.size() * 4, cudaMemcpyHostToDevice));
+    return ZL_OK;
+}
+
 }  // namespace zl

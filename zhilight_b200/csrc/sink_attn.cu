@@ -7,6 +7,7 @@
 // gets dist_bias[h][min(pos - key, n_dist - 1)] added after the scale.  Two more options: no sink at all (an ordinary
 // softmax), and an output rotation: values that were cached turned by their own position give a sum that is turned back
 // by the query's position, pair by pair from a (cos, sin) table, in fp32 before the store.
+// Scores may be soft-capped (cap tanh(s / cap)) and lowered by a slope per head times the distance, in this order, after the scale.
 // With window > 0 a token sees only the last `window` keys up to its own.  Differential attention (MAPS = 2): a query
 // head has two maps, each with queries and keys of its own and its own softmax over the same values; the result is
 // a_1 - lambda a_2 over its root mean square, times a constant, optionally under a full-width sigmoid gate.  Both maps
@@ -78,12 +79,15 @@ __global__ void __launch_bounds__(kSaWarps * 32) k_sink_attn(SinkAttnP p) {
         j_hi = min(pos + 1, j_lo + per);
     }
     const float* bias = p.dist_bias ? p.dist_bias + (size_t)h * p.n_dist : nullptr;
+    const float slope = p.slopes ? p.slopes[h] : 0.f;
     for (int j = j_lo + wm; j < j_hi; j += WPM) {
         const T* kr = kc + (size_t)j * kst;
         float s = 0.f;
         for (int c = lane; c < p.d; c += 32) s = fmaf(sqm[c], to_f32<T>(kr[c]), s);
         s = warp_sum(s);
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
         if (bias) s += bias[min(pos - j, p.n_dist - 1)];
+        if (p.slopes) s = fmaf(-slope, (float)(pos - j), s);
         const float mn = fmaxf(m, s), corr = expf(m - mn), w = expf(s - mn);
         l = fmaf(l, corr, w);
         const T* vr = vc + (size_t)j * vst;
@@ -201,7 +205,8 @@ __device__ __forceinline__ void sa_mma<__nv_bfloat16>(float (&d)[4], const uint3
 // of a key tile with a softmax state of its own; the four states are merged through shared memory at the end.
 // MAPS = 2: the first half of the warps works on the first map, the second on the second; a key tile holds both maps' keys.
 // DEC = false: 32 rows per map.  DEC = true: 16 rows per map, a warp takes 32 of the 64 keys.
-template <typename T, int NV, bool DEC, int MAPS>
+// BIASED: soft cap and slope per head.
+template <typename T, int NV, bool DEC, int MAPS, bool BIASED>
 __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     extern __shared__ __align__(16) unsigned char sa_raw[];
     const SinkAttnP& p = pp.a;
@@ -256,6 +261,8 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     int tok_of[2], pos_of[2], head_of[2], first_of[2];
     bool row_ok[2];
     const float* bias_of[2];
+    float slope_of[2];
+    const float cap_in = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
         const int r = wrow + gq + hh * 8;
@@ -265,6 +272,7 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
         pos_of[hh] = pos0 + tok_of[hh];
         first_of[hh] = sa_first_key(p, pos_of[hh]);
         bias_of[hh] = p.dist_bias ? p.dist_bias + (size_t)(head_of[hh] < p.H ? head_of[hh] : 0) * p.n_dist : nullptr;
+        slope_of[hh] = BIASED && p.slopes ? p.slopes[head_of[hh] < p.H ? head_of[hh] : 0] : 0.f;
     }
     float m_run[2], l_run[2], O[NV][4];
 #pragma unroll
@@ -315,6 +323,7 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
             }
             // scale, mask, online softmax (rows gq and gq + 8 of the warp's 16)
             float mx[2] = {-1e30f, -1e30f};
+            const float dist0[2] = {(float)(pos_of[0] - k0 - kb - 2 * tq), (float)(pos_of[1] - k0 - kb - 2 * tq)};
 #pragma unroll
             for (int j = 0; j < NS; ++j)
 #pragma unroll
@@ -322,6 +331,10 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
                     const int hh = c >> 1, key = k0 + kb + 8 * j + 2 * tq + (c & 1);
                     const bool ok = row_ok[hh] && key < k_hi && key <= pos_of[hh] && key >= first_of[hh];
                     float sc = S[j][c] * p.scale;
+                    if constexpr (BIASED) {
+                        if (p.softcap > 0.f) sc = sa_softcap(sc, p.softcap, cap_in);
+                        sc = fmaf(-slope_of[hh], dist0[hh] - (float)(8 * j + (c & 1)), sc);
+                    }
                     if (ok && bias_of[hh]) sc += bias_of[hh][min(pos_of[hh] - key, p.n_dist - 1)];
                     S[j][c] = ok ? sc : -1e30f;
                     mx[hh] = fmaxf(mx[hh], S[j][c]);
@@ -596,7 +609,7 @@ __global__ void __launch_bounds__(128) k_sink_attn_mma(SinkAttnMmaP pp) {
     }
 }
 
-template <typename T, int NV, bool DEC, int MAPS>
+template <typename T, int NV, bool DEC, int MAPS, bool BIASED>
 static cudaError_t launch_sink_mma(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
     const SinkAttnP& p = pp.a;
     const int qm = DEC ? 16 : kTq / MAPS, nq = qm / (p.H / p.G);
@@ -605,23 +618,23 @@ static cudaError_t launch_sink_mma(const SinkAttnMmaP& pp, int runs, int max_run
     if (!DEC && (p.out_table || MAPS == 2) && smem < (size_t)kTq * (p.vd + 1) * sizeof(float)) smem = (size_t)kTq * (p.vd + 1) * sizeof(float);
     static size_t set_for = 0;
     if (smem > 48 * 1024 && smem > set_for) {
-        const cudaError_t e = cudaFuncSetAttribute(k_sink_attn_mma<T, NV, DEC, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(k_sink_attn_mma<T, NV, DEC, MAPS, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
         set_for = smem;
     }
-    return launch(k_sink_attn_mma<T, NV, DEC, MAPS>, dim3(cdiv(max_run_len, nq), p.G, runs * p.splits), dim3(128), smem, st, pdl, pp);
+    return launch(k_sink_attn_mma<T, NV, DEC, MAPS, BIASED>, dim3(cdiv(max_run_len, nq), p.G, runs * p.splits), dim3(128), smem, st, pdl, pp);
 }
-template <typename T, int NV, int MAPS>
+template <typename T, int NV, int MAPS, bool BIASED>
 static cudaError_t launch_sink_mma_d(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
     // the rows of the longest run fit one 16-row tile: the decode form
-    if (max_run_len * (pp.a.H / pp.a.G) <= 16) return launch_sink_mma<T, NV, true, MAPS>(pp, runs, max_run_len, pdl, st);
-    return launch_sink_mma<T, NV, false, MAPS>(pp, runs, max_run_len, pdl, st);
+    if (max_run_len * (pp.a.H / pp.a.G) <= 16) return launch_sink_mma<T, NV, true, MAPS, BIASED>(pp, runs, max_run_len, pdl, st);
+    return launch_sink_mma<T, NV, false, MAPS, BIASED>(pp, runs, max_run_len, pdl, st);
 }
-template <typename T, int MAPS>
+template <typename T, int MAPS, bool BIASED = false>
 static cudaError_t launch_sink_mma_t(const SinkAttnMmaP& pp, int runs, int max_run_len, bool pdl, cudaStream_t st) {
-    if (pp.a.vd <= 32) return launch_sink_mma_d<T, 4, MAPS>(pp, runs, max_run_len, pdl, st);
-    if (pp.a.vd <= 64) return launch_sink_mma_d<T, 8, MAPS>(pp, runs, max_run_len, pdl, st);
-    return launch_sink_mma_d<T, 16, MAPS>(pp, runs, max_run_len, pdl, st);
+    if (pp.a.vd <= 32) return launch_sink_mma_d<T, 4, MAPS, BIASED>(pp, runs, max_run_len, pdl, st);
+    if (pp.a.vd <= 64) return launch_sink_mma_d<T, 8, MAPS, BIASED>(pp, runs, max_run_len, pdl, st);
+    return launch_sink_mma_d<T, 16, MAPS, BIASED>(pp, runs, max_run_len, pdl, st);
 }
 
 // merge of the splits (at most MS: 4, 8 or 32) with the sink term and the gate; one warp per (token, head), grid
@@ -904,4 +917,34 @@ extern "C" int zl_window_attention(const void* q, void* const* k_addrs, void* co
     }
     ZL_CHECK_CUDA(e);
     return splits > 1 ? sink_attn_merge(p, maps, T, dtype, pdl != 0, stream) : ZL_OK;
+}
+
+extern "C" int zl_biased_sink_attention(const void* q, void* const* k_addrs, void* const* v_addrs, const int32_t* slot,
+                                        const int32_t* pos, const float* sink, int no_sink, float scale, float softcap,
+                                        const float* slopes, int window, void* out, int T, int heads, int kv_heads, int dim, int vdim,
+                                        int splits, void* workspace, size_t workspace_bytes, const int32_t* run_row0,
+                                        const int32_t* run_len, int runs, int max_run_len, int dtype, int pdl, zl_stream_t stream) {
+    ZL_CHECK_ARG(q && k_addrs && v_addrs && slot && pos && out && T > 0 && T <= 65535 && heads > 0 && kv_heads > 0);
+    ZL_CHECK_ARG(heads % kv_heads == 0 && dim > 0 && vdim > 0 && window >= 0 && softcap >= 0.f);
+    ZL_CHECK_SUPPORTED(vdim <= 32 * kSaMaxPerLane && dim <= 2048);
+    ZL_CHECK_ARG(dtype == ZL_F16 || dtype == ZL_BF16 || dtype == ZL_F32);
+    ZL_CHECK_ARG(splits >= 1 && splits <= 32);
+    ZL_CHECK_ARG(splits == 1 || (workspace && workspace_bytes >= zl_sink_attention_workspace_bytes(T, heads, vdim, splits)));
+    SinkAttnP p{q, k_addrs, v_addrs, slot, pos, sink, nullptr, 0, out, heads, kv_heads, dim, vdim, scale, splits,
+                static_cast<float*>(workspace)};
+    p.no_sink = no_sink != 0;
+    p.softcap = softcap;
+    p.slopes = slopes;
+    p.window = window;
+    cudaError_t e;
+    if (sink_mma_eligible(p, run_row0, run_len, runs, max_run_len, 1, dtype)) {
+        ZL_CHECK_ARG((long long)runs * splits <= 65535 && kv_heads <= 65535);
+        SinkAttnMmaP pp{p, run_row0, run_len};
+        e = dtype == ZL_BF16 ? launch_sink_mma_t<__nv_bfloat16, 1, true>(pp, runs, max_run_len, pdl != 0, stream)
+                             : launch_sink_mma_t<__half, 1, true>(pp, runs, max_run_len, pdl != 0, stream);
+    } else if (dtype == ZL_F32) e = launch_sink_general<float, 1>(p, T, pdl != 0, stream);
+    else if (dtype == ZL_BF16) e = launch_sink_general<__nv_bfloat16, 1>(p, T, pdl != 0, stream);
+    else e = launch_sink_general<__half, 1>(p, T, pdl != 0, stream);
+    ZL_CHECK_CUDA(e);
+    return splits > 1 ? sink_attn_merge(p, 1, T, dtype, pdl != 0, stream) : ZL_OK;
 }

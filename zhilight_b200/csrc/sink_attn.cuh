@@ -26,6 +26,8 @@ struct SinkAttnP {
     int out_layout = 0;        // ZL_ROT_HALVES: pair (m, m + vd / 2); ZL_ROT_ADJACENT: pair (2m, 2m + 1)
     int window = 0;            // > 0: keys at distance >= window are not seen
     float lambda = 0.f, out_eps = 0.f, out_mul = 1.f;   // two maps: o = a_1 - lambda a_2, out = out_mul o / sqrt(mean(o^2) + out_eps)
+    float softcap = 0.f;       // > 0: the scaled score s becomes softcap tanh(s / softcap)
+    const float* slopes = nullptr;      // (H): slopes[h] * (pos - key) comes off the score after the cap, or null
     const float* gate_full = nullptr;   // two maps: gate logits, element h * vd + c of row t (row stride ldg), or null
 };
 
@@ -36,6 +38,12 @@ int sink_attn_merge(const SinkAttnP& p, int maps, int T, int dtype, bool pdl, cu
 __device__ __forceinline__ int sa_first_key(const SinkAttnP& p, int pos) {
     if (p.window > 0) return pos >= p.window ? pos - p.window + 1 : 0;
     return p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0;
+}
+
+// softcap tanh(s / softcap) through one exponential: tanh(x) = 1 - 2 / (exp(2 x) + 1).  Its absolute error is a few float ulps of
+// `softcap`, and absolute is what counts in a score; both limits are right (exp overflows to infinity, underflows to 0).
+__device__ __forceinline__ float sa_softcap(float s, float cap, float two_over_cap) {
+    return cap - __fdividef(2.0f * cap, __expf(s * two_over_cap) + 1.0f);
 }
 
 __device__ __forceinline__ void sa_cp_async16(void* smem_dst, const void* gsrc) {

@@ -114,6 +114,16 @@ def _build_dekalorn(config, dtype, max_batch, max_seq, max_step_tokens, **kw):
 register("Dekalorn", _build_dekalorn, ("bfloat16", "float32"))
 
 
+# ---- Bezasun ---------------------------------------------------------------------------------------------------------
+def _build_bezasun(config, dtype, max_batch, max_seq, max_step_tokens, **kw):
+    from .bezasun import BezasunDecoder
+    return BezasunDecoder.from_config_dict(config, dtype=dtype, max_batch=max_batch, max_seq=max_seq,
+                                            max_step_tokens=max_step_tokens, **kw)
+
+
+register("Bezasun", _build_bezasun, ("bfloat16", "float32"))
+
+
 # ---- Llama (HF folder) -----------------------------------------------------------------------------------------------
 _HF_LLAMA_NAMES = [
     (r"^model\.embed_tokens\.weight$", "token_embedding.weight"),
