@@ -938,6 +938,143 @@ def run_compare_dekalorn(args):
                       "clocks": clocks, "timing": "CUDA events on the model's stream; weights per pass larger than L2"}))
 
 
+# ----------------------------------------------------------------------------------------------------------------------
+# --compare-bezasun: prefill and decode throughput of the Bezasun family beside Kodupel (the closest existing model: attention
+# with a sink over slot caches, a recurrent state, silu-like gated experts of three matrices, an fp32 residual) at equal width,
+# depth, heads and feed-forward parameters per token, random weights; --compare-models may add "dekalorn" and "dekipel" (latent
+# attention).  Does not touch the default workload.
+# ----------------------------------------------------------------------------------------------------------------------
+BEZASUN = dict(streams=4, kv_rank=512, rot=64, window=1024, state=128, groups=8, vdim=64, conv=4)
+
+
+def _bezasun_config(sz):
+    """Layers: state space, attention, latent attention, state space; experts everywhere, one of them shared by all tokens."""
+    H, d, D, Z = sz["heads"], sz["dim"], sz["width"], BEZASUN
+    moe = {"kind": "moe", "expert": {"ff": sz["ff_e"]}, "router": {"experts": sz["experts"], "top": sz["top"] - 1},
+           "shared": {"ff": sz["ff_e"]}}
+    ssm = {"type": "mamba2", "mixer": dict(heads=2 * D // Z["vdim"], vdim=Z["vdim"], state=Z["state"], groups=Z["groups"],
+                                           conv=Z["conv"], norm_groups=Z["groups"])}
+    att = {"type": "attention", "mixer": dict(heads=H, kv_heads=8, dim=d, vdim=d, scale=d ** -0.5, softcap=30.0,
+                                              q_temp={"coef": 0.1, "every": 1024})}
+    latent = {"type": "latent_attention",
+              "mixer": dict(heads=H, dim=d, rot_dim=Z["rot"], vdim=d, q_rank=3 * D // 8, kv_rank=Z["kv_rank"],
+                            scale=(d + Z["rot"]) ** -0.5, mask={"size": Z["window"]},
+                            rot={"base": 1e4, "dims": Z["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})}
+    kinds = (ssm, att, latent, ssm)
+    return {"architecture": "Bezasun", "vocab": sz["vocab"], "width": D, "streams": Z["streams"], "residual_mult": 1.0, "logit_scale": 1.0,
+            "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": [dict(kinds[i % 4], mlp=moe) for i in range(sz["layers"])]}
+
+
+def _bezasun_params(sz, rows, ctx):
+    """(Linear parameters one token uses, parameters a step of `rows` tokens reads, cache bytes a token at `ctx` reads plus
+    state bytes it reads and writes)."""
+    D, H, d, E, top, fe, Z = sz["width"], sz["heads"], sz["dim"], sz["experts"], sz["top"] - 1, sz["ff_e"], BEZASUN
+    R, r, Q = Z["kv_rank"], Z["rot"], 3 * D // 8
+    touched = E * (1.0 - (1.0 - top / E) ** rows)
+    inner, bc, hs = 2 * D, Z["groups"] * Z["state"], 2 * D // Z["vdim"]
+    mix = {0: D * (2 * inner + 2 * bc + hs) + inner * D, 1: D * (H * d + 2 * 8 * d) + H * d * D,
+           2: D * (Q + R + r) + Q * H * (d + r) + 2 * H * d * R + H * d * D}
+    moved = {0: 2 * inner * Z["state"] * 4, 1: ctx * 2 * 8 * d * 2, 2: min(ctx, Z["window"]) * (R + r) * 2}
+    active = read = sz["vocab"] * D
+    cache = 0
+    for i in range(sz["layers"]):
+        k = (0, 1, 2, 0)[i % 4]
+        active += mix[k] + E * D + (top + 1) * 3 * D * fe
+        read += mix[k] + E * D + (touched + 1) * 3 * D * fe
+        cache += moved[k]
+    return active, read, cache
+
+
+def run_compare_bezasun(args):
+    import numpy as np
+    import torch
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: the hot path has no CPU fallback")
+    torch.cuda.set_device(0)
+    from zhilight_b200 import build
+    build.build()
+    from zhilight_b200.bezasun import BezasunDecoder
+    from zhilight_b200.dekalorn import DekalornDecoder
+    from zhilight_b200.dekipel import DekipelDecoder
+    from zhilight_b200.kodupel import KodupelDecoder
+    hbm, how = read_peaks()
+    peaks_path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = json.load(open(peaks_path))["bf16_tflops"] if os.path.exists(peaks_path) else 1590.0
+    ctx, chunk, n_prompt = args.prompt if args.prompt > 128 else 1024, 1024, 2048
+    steps, warm = max(args.steps, 16), max(args.warmup, 3)
+    rng = np.random.default_rng(0)
+    rows = []
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.mark_region_start()
+    for name, sz in KODUPEL_SIZES.items():
+        if args.compare_sizes and name not in args.compare_sizes.split(","):
+            continue
+        for kind in [k for k in ("bezasun", "kodupel", "dekalorn", "dekipel") if k in args.compare_models.split(",")]:
+            max_seq = max(ctx, n_prompt) + 4 * (steps + warm) + 64
+            kw = dict(dtype="bf16", max_batch=32, max_seq=max_seq, max_step_tokens=chunk, use_pdl=not args.no_pdl,
+                      use_graph=not args.no_graph)
+            if kind == "bezasun":
+                dec = BezasunDecoder.from_config_dict(_bezasun_config(sz), **kw)
+                active = _bezasun_params(sz, 1, ctx)[0]
+            elif kind == "dekalorn":
+                dec = DekalornDecoder.from_config_dict(_dekalorn_config(sz), **kw)
+                active = _dekalorn_params(sz, 1, ctx)[0]
+            elif kind == "kodupel":
+                dec = KodupelDecoder.from_config_dict(_kodupel_config(sz), **kw)
+                active = _kodupel_params(sz, 1)[0]
+            else:
+                dec = DekipelDecoder.from_config_dict(_dekipel_config(COMPARE_SIZES[name]), **kw)
+                active = _linear_params("dekipel", COMPARE_SIZES[name])
+            dec.init_synthetic(seed=1)
+            stream = torch.cuda.ExternalStream(dec.stream())
+            out = {"size": name, "model": kind}
+            toks = rng.integers(0, sz["vocab"], n_prompt).astype(np.int32)
+            for _ in range(2):
+                dec.prefill(0, toks, 0)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(stream)
+            for _ in range(3):
+                dec.prefill(0, toks, 0)
+            e1.record(stream)
+            e1.synchronize()
+            ms = e0.elapsed_time(e1) / 3
+            out["linear_params_per_token"] = int(active)
+            flops = 2.0 * (active - sz["vocab"] * sz["width"]) * n_prompt
+            out["prefill"] = {"tokens": n_prompt, "chunk": chunk, "ms": round(ms, 3), "tok_s": round(n_prompt / ms * 1e3),
+                              "linear_tflops": round(flops / ms / 1e9, 1),
+                              "of_measured_bf16_peak": round(flops / ms / 1e9 / tflops, 4)}
+            for b in range(32):
+                dec.prefill(b, toks[:ctx], 0)
+            for B in (1, 32):
+                dec.set_state(rng.integers(0, sz["vocab"], B).astype(np.int32), np.full(B, ctx, dtype=np.int32))
+                ms, _ = measure_decode(dec, B, steps, warm, stream, torch.cuda.synchronize)
+                mid = ctx + warm + steps // 2
+                if kind == "bezasun":
+                    _, read, cache = _bezasun_params(sz, B, mid)
+                    step_bytes = read * 2 + B * cache
+                elif kind == "dekalorn":
+                    _, read, cache = _dekalorn_params(sz, B, mid)
+                    step_bytes = read * 2 + B * cache
+                elif kind == "kodupel":
+                    _, read, cache, state = _kodupel_params(sz, B)
+                    step_bytes = read * 2 + B * (mid * cache + state)
+                else:
+                    step_bytes = active * 2 + B * mid * COMPARE_SIZES[name]["kv_rank"] * 2 * ((sz["layers"] + 1) // 2)
+                out["decode_b%d" % B] = {"ctx": ctx, "ms_per_step": round(ms / steps, 4), "tok_s": round(B * steps / ms * 1e3, 1),
+                                          "step_bytes": int(step_bytes),
+                                          "of_%s_hbm_peak" % how: round(step_bytes / (ms / steps * 1e-3) / 1e9 / hbm, 4)}
+            out["kernels_per_step"] = dec.stats()[1]
+            dec.close()
+            del dec
+            torch.cuda.empty_cache()
+            rows.append(out)
+            print(json.dumps(out), file=sys.stderr, flush=True)
+    clocks = sampler.finish()
+    print(json.dumps({"compare": "bezasun vs %s (bf16, random weights, synthetic tokens)" % args.compare_models, "rows": rows,
+                      "clocks": clocks, "timing": "CUDA events on the model's stream; weights per pass larger than L2"}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -970,6 +1107,8 @@ def main():
                     help="instead of the default workload: Dizizen beside Kodupel at a few layer sizes")
     ap.add_argument("--compare-dekalorn", action="store_true",
                     help="instead of the default workload: Dekalorn beside Kodupel at a few layer sizes")
+    ap.add_argument("--compare-bezasun", action="store_true",
+                    help="instead of the default workload: Bezasun beside Kodupel at a few layer sizes")
     ap.add_argument("--compare-dekipel", action="store_true",
                     help="instead of the default workload: Dekipel beside the bf16 Llama decoder at a few layer sizes")
     args = ap.parse_args()
@@ -985,6 +1124,11 @@ def main():
         if args.compare_models == "dekipel,llama":
             args.compare_models = "dekalorn,kodupel"
         run_compare_dekalorn(args)
+        return
+    if args.compare_bezasun:
+        if args.compare_models == "dekipel,llama":
+            args.compare_models = "bezasun,kodupel"
+        run_compare_bezasun(args)
         return
     if args.compare_lagelorn:
         if args.compare_models == "dekipel,llama":

@@ -230,3 +230,49 @@ def forward(cfg, W, tokens):
         kept.append(c)
     out = rms(x.sum(axis=0), cfg.norm_eps) * (1.0 + W["final.norm"])
     return (out @ W["head"].T) * cfg.logit_scale, np.stack(per_layer), kept
+
+
+def bf16_round(a):
+    """float32 array rounded to the nearest bfloat16 (ties to even), still float32."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32).astype(np.uint64)
+    u = (u + 0x7FFF + ((u >> 16) & 1)) & 0xFFFF0000
+    return u.astype(np.uint32).view(np.float32).reshape(np.shape(a))
+
+
+def random_weights(cfg, seed=0, router_gain=3.0):
+    """name -> float32 array whose values are exact in bfloat16.  Router rows are scaled up so that the choice of experts
+    does not hang on a rounding; queries and keys so that attention is not flat; the state-space step sizes so that some
+    heads forget within a few tokens and some remember hundreds; the streams mix differently in every sublayer."""
+    rng = np.random.default_rng(seed)
+    W = {}
+    for name, shp in sorted(cfg.tensor_shapes().items()):
+        last = name.rsplit(".", 1)[-1]
+        norm = rng.standard_normal(shp)
+        if last in ("norm1", "norm2") or name == "final.norm":
+            a = 0.2 * norm
+        elif name.endswith(("q.norm", "k.norm")):
+            a = 1.2 + 0.2 * norm
+        elif last == "norm":
+            a = 1.0 + 0.2 * norm
+        elif ".hc" in name:
+            a = np.eye(shp[0]) * 0.8 + 0.2 * norm if last == "mix" else (0.5 + 0.3 * norm if last == "out" else 1.0 / shp[0] + 0.3 * norm)
+        elif last in ("sink", "D"):
+            a = 0.5 + norm
+        elif last == "A_log":
+            a = rng.uniform(-2.0, 1.0, shp)
+        elif last == "dt_bias":
+            a = rng.uniform(-5.0, 0.5, shp)
+        elif name == "embed":
+            a = 0.12 * norm
+        elif last == "b":
+            a = 0.2 * norm
+        elif last == "conv":
+            a = norm / math.sqrt(shp[-1])
+        elif last == "router":
+            a = router_gain * norm / math.sqrt(shp[-1])
+        elif last in ("uq", "uk"):
+            a = 1.3 * norm / math.sqrt(shp[-1])
+        else:
+            a = norm / math.sqrt(shp[-1])
+        W[name] = bf16_round(a.astype(np.float32))
+    return W

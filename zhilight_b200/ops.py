@@ -913,3 +913,110 @@ def latent_attention_ex(q_absorbed, cache, table, slot, pos, scale, rank_cols, s
               gate.shape[1] if gate is not None else 0, scale, _p(out), t, h, rank_cols, rs, splits, _p(ws), nbytes, _p(run_row0),
               _p(run_len), run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(cache), 0, _stream())
     return out
+
+
+# ------------------------------------------------------------------ hyper-connected streams, biased sink attention, latent
+# attention in a window, selective state space
+def rope_table_scaled(pos, inv_freq, mult):
+    """rope_table with cos and sin times mult."""
+    t, half = pos.numel(), inv_freq.numel()
+    out = torch.empty((t, half, 2), dtype=torch.float32, device=pos.device)
+    _lib.call("zl_rope_table_scaled", _p(pos), t, ctypes.cast(_p(inv_freq), ctypes.POINTER(ctypes.c_double)), half, mult, _p(out), 0,
+              _stream())
+    return out
+
+
+def qkv_headnorm_append_ex(proj, q_off, k_off, v_off, heads, kv_heads, dim, vdim, q_weight, k_weight, k_slots, v_slots, slot, pos, dtype,
+                           eps, value_norm=False, temp_coef=0.0, temp_every=1.0):
+    """proj (T, ld) fp32 -> q (T, heads * dim) of `dtype`: normed per head, times the query temperature of its position; normed keys
+    and values (value_norm: of unit RMS, else as projected) go to rows (slot, pos) of the caches behind the slot tables."""
+    t, ldp = proj.shape
+    q = torch.empty((t, heads * dim), dtype=dtype, device=proj.device)
+    _lib.call("zl_qkv_headnorm_append_ex", _p(proj), ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, _p(q_weight), _p(k_weight),
+              int(value_norm), temp_coef, float(temp_every), None, 0, 1.0, eps, _p(q), _p(k_slots), _p(v_slots), _p(slot), _p(pos), t,
+              _dt(q), 0, _stream())
+    return q
+
+
+def biased_sink_attention(q, k_table, v_table, slot, pos, scale, heads, kv_heads, dim, vdim, sink=None, no_sink=False, softcap=0.0,
+                          slopes=None, window=0, splits=1, run_row0=None, run_len=None, max_run_len=0):
+    """Attention with soft-capped scores, a slope per head (fp32 (heads) or None) times the distance taken off, and a sink."""
+    t = q.shape[0]
+    nbytes = _lib.load().zl_sink_attention_workspace_bytes(t, heads, vdim, splits)
+    ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=q.device)
+    out = torch.empty((t, heads * vdim), dtype=q.dtype, device=q.device)
+    _lib.call("zl_biased_sink_attention", _p(q), _p(k_table), _p(v_table), _p(slot), _p(pos), _p(sink), int(no_sink), scale, softcap,
+              _p(slopes), window, _p(out), t, heads, kv_heads, dim, vdim, splits, _p(ws), nbytes, _p(run_row0), _p(run_len),
+              run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(q), 0, _stream())
+    return out
+
+
+def latent_rope_append_split(q_proj, heads, dim, rot_dim, table, kv_proj, c_off, kv_rank, kv_weight, rank_cols, qa, cache, slot_tab,
+                             slot, pos, eps):
+    """latent_rope_append with the queries (T, heads * (dim + rot_dim)) in a matrix of their own."""
+    t = q_proj.shape[0]
+    q = torch.empty((t, heads, dim), dtype=cache.dtype, device=q_proj.device)
+    _lib.call("zl_latent_rope_append_split", _p(q_proj), q_proj.shape[1], heads, dim, rot_dim, _p(table), _p(q), _p(qa), _p(kv_proj),
+              kv_proj.shape[1], c_off, kv_rank, _p(kv_weight), rank_cols, cache.shape[2], _p(slot_tab), _p(slot), _p(pos), t, eps,
+              _dt(cache), 0, _stream())
+    return q
+
+
+def latent_window_attention(q_absorbed, cache, table, slot, pos, scale, rank_cols, window, sink=None, gate=None, splits=1,
+                            run_row0=None, run_len=None, max_run_len=0):
+    """latent_attention_ex in a sliding window of `window` rows (0: none)."""
+    t, h, rs = q_absorbed.shape
+    lib = _lib.load()
+    _lib.check(lib.zl_latent_attention_prepare_ex(h, rank_cols, rs, _dt(cache)))
+    nbytes = lib.zl_latent_attention_workspace_bytes(t, h, rank_cols, splits)
+    ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=cache.device)
+    out = torch.empty((t, h, rank_cols), dtype=cache.dtype, device=cache.device)
+    _lib.call("zl_latent_window_attention", _p(q_absorbed), _p(table), _p(slot), _p(pos), _p(sink), _p(gate),
+              gate.shape[1] if gate is not None else 0, scale, window, _p(out), t, h, rank_cols, rs, splits, _p(ws), nbytes, _p(run_row0),
+              _p(run_len), run_row0.numel() if run_row0 is not None else 0, max_run_len, _dt(cache), 0, _stream())
+    return out
+
+
+def hyper_update(x, parts, mix, out, w_in=None, coef=None, dense=None, next_w=None, want_u=False, eps=1e-6, act_dtype=torch.float32):
+    """x (T, S, D) fp32 in place: x_s' <- sum_s mix[s, s'] x_s + out[s'] y with y = sum_p coef[:, p] parts[:, p] + dense (parts
+    (T, P, D) fp32 or None: no update); u = sum_s w_in[s] x_s (None: the sum).  -> (next_w * rms(u) of act_dtype or None, u or None)."""
+    t, s, d = x.shape
+    h = torch.empty((t, d), dtype=act_dtype, device=x.device) if next_w is not None else None
+    u = torch.empty((t, d), dtype=torch.float32, device=x.device) if want_u else None
+    code = {torch.float16: F16, torch.bfloat16: BF16, torch.float32: F32}[act_dtype]
+    _lib.call("zl_hyper_update", _p(x), s, _p(parts), d, _p(coef), parts.shape[1] if parts is not None else 0, _p(dense), d, _p(mix),
+              _p(out), _p(w_in), _p(next_w), _p(h), _p(u), code, t, d, eps, 0, _stream())
+    return h, u
+
+
+def hyper_embed(ids, table, scale, streams, w_in=None, next_w=None, want_u=False, eps=1e-6):
+    """-> (x (T, streams, D) fp32, next_w * rms(sum_s w_in[s] x_s) in the table's dtype or None, that sum or None)."""
+    t, d = ids.numel(), table.shape[1]
+    x = torch.empty((t, streams, d), dtype=torch.float32, device=table.device)
+    h = torch.empty((t, d), dtype=table.dtype, device=table.device) if next_w is not None else None
+    u = torch.empty((t, d), dtype=torch.float32, device=table.device) if want_u else None
+    _lib.call("zl_hyper_embed", _p(ids), _p(table), table.shape[0], scale, _p(x), streams, _p(w_in), _p(next_w), _p(h), _p(u), _dt(table),
+              t, d, eps, 0, _stream())
+    return x, h, u
+
+
+def ssm_scan(proj, col_x, col_dt, conv_weight, conv_bias, dt_bias, a_log, d_skip, ring_table, run_row0, run_len, slot, pos, state_table,
+             heads, vdim, state, groups):
+    """proj (T, ld) fp32, conv_weight (taps, channels) fp32 -> o (T, heads * vdim) fp32; states and rings behind the slot tables are
+    read and written."""
+    t, ld = proj.shape
+    o = torch.empty((t, heads * vdim), dtype=torch.float32, device=proj.device)
+    nbytes = _lib.load().zl_ssm_workspace_bytes(t, heads, vdim, state, groups)
+    ws = torch.empty(nbytes, dtype=torch.uint8, device=proj.device)
+    _lib.call("zl_ssm_scan", _p(proj), ld, col_x, col_dt, _p(conv_weight), _p(conv_bias), conv_weight.shape[0], _p(dt_bias), _p(a_log),
+              _p(d_skip), _p(ring_table), _p(run_row0), _p(run_len), run_row0.numel(), _p(slot), _p(pos), _p(state_table), _p(o),
+              heads * vdim, heads, vdim, state, groups, t, _p(ws), nbytes, 0, _stream())
+    return o
+
+
+def silu_gate_group_rmsnorm(o, z, weight, groups, eps, out_dtype):
+    """weight * rms over equal parts of o * silu(z); o (T, D) fp32, z (T, >= D) fp32 (its first D columns)."""
+    t, d = o.shape
+    y = torch.empty((t, d), dtype=out_dtype, device=o.device)
+    _lib.call("zl_silu_gate_group_rmsnorm", _p(o), d, _p(z), z.shape[1], _p(weight), _p(y), d, t, d, groups, eps, _dt(y), 0, _stream())
+    return y
