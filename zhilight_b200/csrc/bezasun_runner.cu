@@ -229,7 +229,8 @@ int len_bucket(const zl_bezasun* m, int max_len) {
 int attn_splits(const BLayer& L, int T, int max_len) {
     const auto& lc = L.c;
     if (lc.type == ZL_BEZASUN_LATENT)
-        return zl_latent_attention_splits(T, lc.heads, L.rank_cols, lc.window > 0 && lc.window < max_len ? lc.window : max_len);
+        // (a window is full, a length bucket is not: splits half as long)
+        return zl_latent_attention_splits(T, lc.heads, L.rank_cols, lc.window > 0 && lc.window < max_len / 2 ? 2 * lc.window : max_len);
     return lc.type == ZL_BEZASUN_ATTENTION ? zl_sink_attention_splits(T, lc.heads, lc.kv_heads, max_len) : 1;
 }
 

@@ -6,11 +6,11 @@
 // k_ssm_prep: convolution, silu, step sizes and decays of all rows of the step at once.  k_ssm_scan: a row of S (one value
 // channel) depends on its own past and the token's vectors only; it is walked through the tokens of its sequence in order, so a
 // token's result does not depend on how the sequence was cut into steps or on the rest of the step.  A CTA owns 32 channels of
-// one head of one run; a channel's state lives in the registers of four adjacent lanes, in 4-element pieces f = 4 i + q of the
-// state dimension (their 16-byte reads of a staged vector fall into different banks), updated and read out with packed fp32
-// pairs.  The token vectors fly into shared memory chunk by chunk ahead of use.  State sizes above 256 take k_ssm_scan_any
-// (state in shared memory, one thread per channel).  A run that starts at position 0 starts from a zero state (a slot given to
-// a new sequence needs no clearing); the final state and the convolution's last inputs go back to the slot.
+// one head of one run; two channels' states live in the registers of eight adjacent lanes, in 4-element pieces f = 8 i + q of the
+// state dimension, updated and read out with packed fp32 pairs.  The token vectors fly into shared memory chunk by chunk ahead
+// of use.  k_ssm_step: the same for one token per sequence, straight from and to the states.  State sizes above 256 take
+// k_ssm_scan_any (state in shared memory, one thread per channel).  A run that starts at position 0 starts from a zero state (a
+// slot given to a new sequence needs no clearing); the final state and the convolution's last inputs go back to the slot.
 #include "common.cuh"
 
 namespace zl {
@@ -33,18 +33,39 @@ struct SsmP {
     int vec;                    // staged pieces of 16 bytes
 };
 
-constexpr int kSsChunk = 16, kSsCols = 32, kSsLanes = 4, kSsThreads = kSsCols * kSsLanes;
+constexpr int kSsChunk = 16, kSsCols = 32, kSsThreads = 128;
 
 __device__ __forceinline__ float ss_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
-// grid (channel blocks + 1, T); the last block computes the heads' step sizes.  V channels per thread (4: 16-byte rows).
 template <int V>
-__global__ void __launch_bounds__(256) k_ssm_prep(SsmP p) {
+struct SsVec {
+    float v[V];
+};
+template <int V>
+__device__ __forceinline__ SsVec<V> ss_load(const float* p) {
+    SsVec<V> r;
+    if constexpr (V == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        r.v[0] = a.x, r.v[1] = a.y, r.v[2] = a.z, r.v[3] = a.w;
+    } else {
+        r.v[0] = p[0];
+    }
+    return r;
+}
+
+// grid (channel blocks + 1, ceil(T / ROWS)); the last block computes the heads' step sizes.  V channels per thread (4: 16-byte
+// rows).  TAPS > 0: that many taps, a thread's rows and the ones before them are loaded once, all in flight; 0: any number, read
+// back row by row.  An earlier input is a row of this step if that belongs to the same sequence, else the slot's ring, else
+// (before the start) zero.
+template <int V, int TAPS, int ROWS>
+__global__ void __launch_bounds__(256) k_ssm_prep(SsmP p, int T) {
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.y, sl = p.slot[t], pos = p.pos[t], nr = p.taps - 1, C = p.C;
+    constexpr int NR = TAPS > 0 ? TAPS - 1 : 0;
+    const int t0 = blockIdx.y * ROWS, rows = min(ROWS, T - t0), nr = TAPS > 0 ? NR : p.taps - 1, C = p.C;
     if (blockIdx.x == gridDim.x - 1) {
-        for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
+        for (int i = threadIdx.x; i < rows * p.H; i += blockDim.x) {
+            const int t = t0 + i / p.H, h = i % p.H;
             const float dt = ss_softplus(p.proj[(size_t)t * p.ld + p.col_dt + h] + p.dt_bias[h]);
             p.dtd[(size_t)t * p.H + h] = make_float2(dt, expf(-expf(p.a_log[h]) * dt));
         }
@@ -52,32 +73,63 @@ __global__ void __launch_bounds__(256) k_ssm_prep(SsmP p) {
     }
     const int c = (blockIdx.x * 256 + threadIdx.x) * V;
     if (c >= C) return;
-    const float* row = p.proj + (size_t)t * p.ld + p.col_x + c;
-    const float* ring = nr > 0 ? static_cast<const float*>(p.ring_addrs[sl]) + c : nullptr;
-    // how many earlier rows of this step belong to the same sequence (at most taps - 1 matter)
-    int back = 0;
-    while (back < nr && t - back - 1 >= 0 && p.slot[t - back - 1] == sl) ++back;
-    float acc[V];
+    const float* src = p.proj + p.col_x + c;
+    const SsVec<V> bias = ss_load<V>(p.conv_b + c);
+    SsVec<V> w[TAPS > 0 ? TAPS : 1], x[NR + ROWS];   // x[NR + i]: row t0 + i
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = p.conv_b[c + i];
-    auto add = [&](const float* w, const float* x) {
-        if constexpr (V == 4) {
-            const float4 a = *reinterpret_cast<const float4*>(w), b = *reinterpret_cast<const float4*>(x);
-            acc[0] = fmaf(a.x, b.x, acc[0]), acc[1] = fmaf(a.y, b.y, acc[1]), acc[2] = fmaf(a.z, b.z, acc[2]), acc[3] = fmaf(a.w, b.w, acc[3]);
-        } else {
-            acc[0] = fmaf(w[0], x[0], acc[0]);
-        }
-    };
-    add(p.conv_w + (size_t)nr * C + c, row);
-#pragma unroll 3
-    for (int j = 1; j <= nr; ++j) {   // the input j positions back
-        const int pj = pos - j;
-        if (pj < 0) break;
-        add(p.conv_w + (size_t)(nr - j) * C + c, j <= back ? row - (long long)j * p.ld : ring + (size_t)(pj % nr) * C);
+    for (int j = 0; j < TAPS; ++j) w[j] = ss_load<V>(p.conv_w + (size_t)j * C + c);
+#pragma unroll
+    for (int i = 0; i < NR + ROWS; ++i) {
+        const int t = t0 + i - NR;
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[i].v[e] = 0.f;
+        if (t >= 0 && t < T) x[i] = ss_load<V>(src + (size_t)t * p.ld);
     }
-    float* dst = p.xbc + (size_t)t * C + c;
-    if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(silu_f(acc[0]), silu_f(acc[1]), silu_f(acc[2]), silu_f(acc[3]));
-    else dst[0] = silu_f(acc[0]);
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        if (i >= rows) break;
+        const int t = t0 + i, sl = p.slot[t], pos = p.pos[t];
+        int back = 0;   // how many earlier rows of this step belong to the same sequence (at most taps - 1 matter)
+        while (back < nr && t - back - 1 >= 0 && p.slot[t - back - 1] == sl) ++back;
+        SsVec<V> acc = bias;
+        auto add = [&](const SsVec<V>& a, const SsVec<V>& v) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) acc.v[e] = fmaf(a.v[e], v.v[e], acc.v[e]);
+        };
+        auto stored = [&](int j) { return ss_load<V>(static_cast<const float*>(p.ring_addrs[sl]) + (size_t)((pos - j) % nr) * C + c); };
+        if constexpr (TAPS > 0) {
+            add(w[NR], x[NR + i]);
+#pragma unroll
+            for (int j = 1; j <= NR; ++j) {
+                if (j <= back) add(w[NR - j], x[NR + i - j]);
+                else if (pos >= j) add(w[NR - j], stored(j));
+            }
+        } else {
+            add(ss_load<V>(p.conv_w + (size_t)nr * C + c), x[i]);
+            for (int j = 1; j <= nr && j <= pos; ++j)
+                add(ss_load<V>(p.conv_w + (size_t)(nr - j) * C + c), j <= back ? ss_load<V>(src + (size_t)(t - j) * p.ld) : stored(j));
+        }
+        float* dst = p.xbc + (size_t)t * C + c;
+        if constexpr (V == 4)
+            *reinterpret_cast<float4*>(dst) = make_float4(silu_f(acc.v[0]), silu_f(acc.v[1]), silu_f(acc.v[2]), silu_f(acc.v[3]));
+        else
+            dst[0] = silu_f(acc.v[0]);
+    }
+}
+
+template <int V, int ROWS>
+static cudaError_t ssm_prep_launch(const SsmP& p, int T, bool pdl, cudaStream_t st) {
+    const dim3 grid(cdiv(p.C, 256 * V) + 1, cdiv(T, ROWS)), block(256);
+    switch (p.taps) {
+        case 2: return launch(k_ssm_prep<V, 2, ROWS>, grid, block, 0, st, pdl, p, T);
+        case 3: return launch(k_ssm_prep<V, 3, ROWS>, grid, block, 0, st, pdl, p, T);
+        case 4: return launch(k_ssm_prep<V, 4, ROWS>, grid, block, 0, st, pdl, p, T);
+        default: return launch(k_ssm_prep<V, 0, ROWS>, grid, block, 0, st, pdl, p, T);
+    }
+}
+template <int V>
+static cudaError_t ssm_prep_launch(const SsmP& p, int T, bool pdl, cudaStream_t st) {
+    return T > 64 ? ssm_prep_launch<V, 4>(p, T, pdl, st) : ssm_prep_launch<V, 1>(p, T, pdl, st);
 }
 
 // packed pairs of fp32
@@ -120,28 +172,37 @@ __device__ __forceinline__ void ss_store_tails(const SsmP& p, int row0, int len,
     }
 }
 
-// grid (ceil(dv / 32), H, runs).  P: pieces per lane, the state is at most 16 P long.
-template <int P>
+// grid (ceil(dv / 32), H, runs).  LANES adjacent lanes share CE channels: a lane holds P pieces of each of them (the state is at
+// most 4 P LANES long), so that a staged piece of B or C serves CE channels.
+template <int P, int LANES, int CE>
 __global__ void __launch_bounds__(kSsThreads) k_ssm_scan(SsmP p) {
-    constexpr int NP = P * kSsLanes * 4, PER = 2 * NP + kSsCols + 4;   // staged per token: B | C | x | dt, decay
+    static_assert(kSsThreads / LANES * CE == kSsCols && 4 * CE == LANES, "a lane per (token, channel) of a group of four tokens");
+    constexpr int NP = P * LANES * 4, PER = 2 * NP + kSsCols + 4;   // staged per token: B | C | x | dt, decay
     extern __shared__ __align__(16) float ssm[];   // [2][kSsChunk][PER]
     pdl_trigger();
     pdl_wait();
     const int run = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, N = p.N;
     const int row0 = p.run_row0[run], len = p.run_len[run];
     if (len <= 0) return;
-    const int q = tid & (kSsLanes - 1), col = tid / kSsLanes, j0 = blockIdx.x * kSsCols, j = j0 + col;
-    const bool mine = j < p.dv;   // the lanes of a channel agree
+    const int q = tid & (LANES - 1), col = tid / LANES * CE, j0 = blockIdx.x * kSsCols, j = j0 + col;
     const int sl = p.slot[row0];
     const int inner = p.H * p.dv, g = h / (p.H / p.G), ncol = min(kSsCols, p.dv - j0);
     const float* sB = p.xbc + (size_t)row0 * p.C + inner + (size_t)g * N;
     const float* sX = p.xbc + (size_t)row0 * p.C + (size_t)h * p.dv + j0;
     const size_t c_off = (size_t)p.G * N;   // from a group's B to its C
-    if (NP > N) {   // padding of the staged vectors: zero, never written again
+    // padding of the staged vectors: zero, never written again
+    if (NP > N) {
         const int pad = NP - N;
         for (int i = tid; i < 2 * kSsChunk * 2 * pad; i += kSsThreads) {
             const int v = i / pad, e = i - v * pad;   // v: (buffer, token, B or C)
             ssm[(size_t)(v >> 1) * PER + (v & 1) * NP + N + e] = 0.f;
+        }
+    }
+    if (ncol < kSsCols) {
+        const int pad = kSsCols - ncol;
+        for (int i = tid; i < 2 * kSsChunk * pad; i += kSsThreads) {
+            const int v = i / pad, e = i - v * pad;
+            ssm[(size_t)v * PER + 2 * NP + ncol + e] = 0.f;
         }
     }
     auto stage = [&](int buf, int c0) {
@@ -166,28 +227,61 @@ __global__ void __launch_bounds__(kSsThreads) k_ssm_scan(SsmP p) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
-    float* sg = static_cast<float*>(p.state_addrs[sl]) + ((size_t)h * p.dv + (mine ? j : 0)) * N;
+    float* sg = static_cast<float*>(p.state_addrs[sl]) + ((size_t)h * p.dv + j) * N;
     const bool fresh = p.pos[row0] == 0, n4 = (N & 3) == 0;
-    f2 S[2 * P];
+    f2 S[CE][2 * P];
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
-        const int k = (kSsLanes * i + q) * 4;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (mine && !fresh) {
-            if (n4) {
-                if (k < N) v = *reinterpret_cast<const float4*>(sg + k);
-            } else {
-                if (k < N) v.x = sg[k];
-                if (k + 1 < N) v.y = sg[k + 1];
-                if (k + 2 < N) v.z = sg[k + 2];
-                if (k + 3 < N) v.w = sg[k + 3];
+    for (int c = 0; c < CE; ++c)
+#pragma unroll
+        for (int i = 0; i < P; ++i) {
+            const int k = (LANES * i + q) * 4;
+            const float* src = sg + (size_t)c * N + k;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (j + c < p.dv && !fresh) {
+                if (n4) {
+                    if (k < N) v = *reinterpret_cast<const float4*>(src);
+                } else {
+                    if (k < N) v.x = src[0];
+                    if (k + 1 < N) v.y = src[1];
+                    if (k + 2 < N) v.z = src[2];
+                    if (k + 3 < N) v.w = src[3];
+                }
             }
+            S[c][2 * i] = f2_pack(v.x, v.y), S[c][2 * i + 1] = f2_pack(v.z, v.w);
         }
-        S[2 * i] = f2_pack(v.x, v.y), S[2 * i + 1] = f2_pack(v.z, v.w);
-    }
     if (p.taps > 1) ss_store_tails(p, row0, len, static_cast<float*>(p.ring_addrs[sl]));
     const float skip = p.d_skip[h];
     float* optr = p.o + (size_t)row0 * p.ld_o + (size_t)h * p.dv + j;
+    // a token's update of the state and this lane's share of the read-outs
+    auto token = [&](const float* tk, float* out) {
+        const float2 dd = *reinterpret_cast<const float2*>(tk + 2 * NP + kSsCols);
+        const f2 d2 = f2_pack(dd.y, dd.y);
+        f2 v2[CE], o0[CE], o1[CE];
+#pragma unroll
+        for (int c = 0; c < CE; ++c) {
+            const float v = dd.x * tk[2 * NP + col + c];
+            v2[c] = f2_pack(v, v);
+            o0[c] = o1[c] = 0ull;
+        }
+        const ulonglong2* mB = reinterpret_cast<const ulonglong2*>(tk) + q;
+        const ulonglong2* mC = reinterpret_cast<const ulonglong2*>(tk + NP) + q;
+#pragma unroll
+        for (int i = 0; i < P; ++i) {
+            const ulonglong2 b = mB[LANES * i], r = mC[LANES * i];
+#pragma unroll
+            for (int c = 0; c < CE; ++c) {
+                S[c][2 * i] = f2_fma(b.x, v2[c], f2_mul(d2, S[c][2 * i]));
+                S[c][2 * i + 1] = f2_fma(b.y, v2[c], f2_mul(d2, S[c][2 * i + 1]));
+                o0[c] = f2_fma(r.x, S[c][2 * i], o0[c]);
+                o1[c] = f2_fma(r.y, S[c][2 * i + 1], o1[c]);
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < CE; ++c) {
+            const float2 a = f2_unpack(o0[c]), b = f2_unpack(o1[c]);
+            out[c] = (a.x + a.y) + (b.x + b.y);
+        }
+    };
     int buf = 0;
     for (int c0 = 0; c0 < len; c0 += kSsChunk, buf ^= 1) {
         const int cn = min(kSsChunk, len - c0);
@@ -195,41 +289,116 @@ __global__ void __launch_bounds__(kSsThreads) k_ssm_scan(SsmP p) {
         __syncthreads();   // this chunk has landed for every thread; the other half is no longer read
         if (c0 + kSsChunk < len) stage(buf ^ 1, c0 + kSsChunk);
         const float* tv = ssm + (size_t)buf * kSsChunk * PER;
-#pragma unroll 2
-        for (int tt = 0; tt < cn; ++tt, tv += PER, optr += p.ld_o) {
-            const float x = mine ? tv[2 * NP + col] : 0.f;
-            const float2 dd = *reinterpret_cast<const float2*>(tv + 2 * NP + kSsCols);
-            const f2 v2 = f2_pack(dd.x * x, dd.x * x), d2 = f2_pack(dd.y, dd.y);
-            const ulonglong2* mB = reinterpret_cast<const ulonglong2*>(tv) + q;
-            const ulonglong2* mC = reinterpret_cast<const ulonglong2*>(tv + NP) + q;
-            f2 o0 = 0ull, o1 = 0ull;
+        int tt = 0;
+        // four tokens at a time: the sums over the lanes are finished together, each round of shuffles halving the values a lane
+        // carries, until lane q holds the one of token q / CE and channel q % CE.  A sum's order is that of the single-token form.
+        for (; tt + 4 <= cn; tt += 4, tv += 4 * PER, optr += 4 * p.ld_o) {
+            float val[LANES];
 #pragma unroll
-            for (int i = 0; i < P; ++i) {
-                const ulonglong2 b = mB[kSsLanes * i], c = mC[kSsLanes * i];
-                S[2 * i] = f2_fma(b.x, v2, f2_mul(d2, S[2 * i]));
-                S[2 * i + 1] = f2_fma(b.y, v2, f2_mul(d2, S[2 * i + 1]));
-                o0 = f2_fma(c.x, S[2 * i], o0);
-                o1 = f2_fma(c.y, S[2 * i + 1], o1);
+            for (int k = 0; k < 4; ++k) token(tv + k * PER, val + k * CE);
+#pragma unroll
+            for (int m = 1; m < LANES; m <<= 1) {
+                const bool up = q & m;
+#pragma unroll
+                for (int i = 0; i < LANES / (2 * m); ++i) {
+                    const float keep = up ? val[2 * i + 1] : val[2 * i], send = up ? val[2 * i] : val[2 * i + 1];
+                    val[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+                }
             }
-            const float2 a = f2_unpack(o0), b = f2_unpack(o1);
-            float out = (a.x + a.y) + (b.x + b.y);
+            const int k = q / CE, c = q % CE;
+            if (j + c < p.dv) optr[k * p.ld_o + c] = fmaf(skip, tv[k * PER + 2 * NP + col + c], val[0]);
+        }
+        for (; tt < cn; ++tt, tv += PER, optr += p.ld_o) {
+            float val[CE];
+            token(tv, val);
 #pragma unroll
-            for (int m = 1; m < kSsLanes; m <<= 1) out += __shfl_xor_sync(0xffffffffu, out, m);
-            if (mine && q == 0) *optr = fmaf(skip, x, out);
+            for (int c = 0; c < CE; ++c) {
+#pragma unroll
+                for (int m = 1; m < LANES; m <<= 1) val[c] += __shfl_xor_sync(0xffffffffu, val[c], m);
+                if (q == c && j + c < p.dv) optr[c] = fmaf(skip, tv[2 * NP + col + c], val[c]);
+            }
         }
     }
-    if (!mine) return;
+#pragma unroll
+    for (int c = 0; c < CE; ++c) {
+        if (j + c >= p.dv) continue;
+#pragma unroll
+        for (int i = 0; i < P; ++i) {
+            const int k = (LANES * i + q) * 4;
+            float* dst = sg + (size_t)c * N + k;
+            const float2 a = f2_unpack(S[c][2 * i]), b = f2_unpack(S[c][2 * i + 1]);
+            if (n4) {
+                if (k < N) *reinterpret_cast<float4*>(dst) = make_float4(a.x, a.y, b.x, b.y);
+            } else {
+                if (k < N) dst[0] = a.x;
+                if (k + 1 < N) dst[1] = a.y;
+                if (k + 2 < N) dst[2] = b.x;
+                if (k + 3 < N) dst[3] = b.y;
+            }
+        }
+    }
+}
+
+// One token per sequence (decode steps): the state is read, updated, read out and written once, every load independent.  Eight
+// lanes per channel in the pieces and the order of sums of k_ssm_scan.  grid (ceil(dv / 16), H, runs)
+template <int P>
+__global__ void __launch_bounds__(128) k_ssm_step(SsmP p) {
+    constexpr int LANES = 8;
+    pdl_trigger();
+    pdl_wait();
+    const int run = blockIdx.z, h = blockIdx.y, N = p.N, q = threadIdx.x & (LANES - 1), j = blockIdx.x * 16 + (threadIdx.x >> 3);
+    if (p.run_len[run] <= 0) return;
+    const int row = p.run_row0[run], sl = p.slot[row], inner = p.H * p.dv, g = h / (p.H / p.G);
+    const bool mine = j < p.dv, fresh = p.pos[row] == 0;
+    const float* xr = p.xbc + (size_t)row * p.C;
+    const float *B = xr + inner + (size_t)g * N, *Cv = B + (size_t)p.G * N;
+    float* sg = static_cast<float*>(p.state_addrs[sl]) + ((size_t)h * p.dv + (mine ? j : 0)) * N;
+    float S[P][4], b[P][4], r[P][4];
 #pragma unroll
     for (int i = 0; i < P; ++i) {
-        const int k = (kSsLanes * i + q) * 4;
-        const float2 a = f2_unpack(S[2 * i]), b = f2_unpack(S[2 * i + 1]);
-        if (n4) {
-            if (k < N) *reinterpret_cast<float4*>(sg + k) = make_float4(a.x, a.y, b.x, b.y);
+        const int k = (LANES * i + q) * 4;
+        if (p.vec) {   // whole pieces
+            const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 s4 = k < N && mine && !fresh ? *reinterpret_cast<const float4*>(sg + k) : z;
+            const float4 b4 = k < N ? *reinterpret_cast<const float4*>(B + k) : z, r4 = k < N ? *reinterpret_cast<const float4*>(Cv + k) : z;
+            S[i][0] = s4.x, S[i][1] = s4.y, S[i][2] = s4.z, S[i][3] = s4.w;
+            b[i][0] = b4.x, b[i][1] = b4.y, b[i][2] = b4.z, b[i][3] = b4.w;
+            r[i][0] = r4.x, r[i][1] = r4.y, r[i][2] = r4.z, r[i][3] = r4.w;
         } else {
-            if (k < N) sg[k] = a.x;
-            if (k + 1 < N) sg[k + 1] = a.y;
-            if (k + 2 < N) sg[k + 2] = b.x;
-            if (k + 3 < N) sg[k + 3] = b.y;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const bool in = k + e < N;
+                S[i][e] = in && mine && !fresh ? sg[k + e] : 0.f;
+                b[i][e] = in ? B[k + e] : 0.f;
+                r[i][e] = in ? Cv[k + e] : 0.f;
+            }
+        }
+    }
+    if (p.taps > 1) ss_store_tails(p, row, 1, static_cast<float*>(p.ring_addrs[sl]));
+    const float2 dd = p.dtd[(size_t)row * p.H + h];
+    const float x = mine ? xr[(size_t)h * p.dv + j] : 0.f, v = dd.x * x;
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < P; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            S[i][e] = fmaf(b[i][e], v, dd.y * S[i][e]);
+            o[e] = fmaf(r[i][e], S[i][e], o[e]);
+        }
+    float out = (o[0] + o[1]) + (o[2] + o[3]);
+#pragma unroll
+    for (int m = 1; m < LANES; m <<= 1) out += __shfl_xor_sync(0xffffffffu, out, m);
+    if (!mine) return;
+    if (q == 0) p.o[(size_t)row * p.ld_o + (size_t)h * p.dv + j] = fmaf(p.d_skip[h], x, out);
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+        const int k = (LANES * i + q) * 4;
+        if (p.vec) {
+            if (k < N) *reinterpret_cast<float4*>(sg + k) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (k + e < N) sg[k + e] = S[i][e];
         }
     }
 }
@@ -265,22 +434,22 @@ __global__ void __launch_bounds__(32) k_ssm_scan_any(SsmP p) {
         for (int k = 0; k < N; ++k) sg[k] = st[k * 32 + lane];
 }
 
-template <int P>
+template <int P, int LANES, int CE>
 static int ssm_launch(const SsmP& p, int runs, bool pdl, cudaStream_t st) {
-    constexpr size_t smem = (size_t)2 * kSsChunk * (2 * P * kSsLanes * 4 + kSsCols + 4) * sizeof(float);
+    constexpr size_t smem = (size_t)2 * kSsChunk * (2 * P * LANES * 4 + kSsCols + 4) * sizeof(float);
     if (smem > 48 * 1024) {
         static bool set = false;
         if (!set) {
-            ZL_CHECK_CUDA(cudaFuncSetAttribute(k_ssm_scan<P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            ZL_CHECK_CUDA(cudaFuncSetAttribute(k_ssm_scan<P, LANES, CE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             set = true;
         }
     }
-    ZL_CHECK_CUDA(launch(k_ssm_scan<P>, dim3(cdiv(p.dv, kSsCols), p.H, runs), dim3(kSsThreads), smem, st, pdl, p));
+    ZL_CHECK_CUDA(launch(k_ssm_scan<P, LANES, CE>, dim3(cdiv(p.dv, kSsCols), p.H, runs), dim3(kSsThreads), smem, st, pdl, p));
     return ZL_OK;
 }
 
-// y[t] = w * v / sqrt(mean(v^2) + eps) in equal parts, v = o silu(z).  grid (groups, T); the first 8 values of a thread stay in
-// registers between the passes.
+// y[t] = w * v / sqrt(mean(v^2) + eps) in equal parts, v = o silu(z).  One CTA per (token, part): grid (groups, T); the first 8
+// values of a thread stay in registers between the passes.
 template <typename TO>
 __global__ void __launch_bounds__(512) k_silu_gate_group_rmsnorm(const float* __restrict__ o, long long ldo,
                                                                  const float* __restrict__ z, long long ldz,
@@ -317,6 +486,58 @@ __global__ void __launch_bounds__(512) k_silu_gate_group_rmsnorm(const float* __
     for (int c = threadIdx.x + 8 * n; c < gs; c += n) yr[c] = from_f32<TO>(orow[c] * silu_f(zr[c]) * r * w[c0 + c]);
 }
 
+// The same with a warp per (token, part) for parts of at most 1024 values in 16-byte pieces: no barrier, every load in flight.
+// grid (ceil(groups / 8), T), 8 warps
+template <typename TO, int PIECES>
+__global__ void __launch_bounds__(256) k_silu_gate_group_rmsnorm_warp(const float* __restrict__ o, long long ldo,
+                                                                      const float* __restrict__ z, long long ldz,
+                                                                      const float* __restrict__ w, TO* __restrict__ y, long long ldy,
+                                                                      int groups, int gs, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    const int g = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, c0 = g * gs;
+    if (g >= groups) return;
+    const float *orow = o + (size_t)blockIdx.y * ldo + c0, *zr = z + (size_t)blockIdx.y * ldz + c0;
+    float4 keep[PIECES];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+        if (c < gs) a = *reinterpret_cast<const float4*>(orow + c), b = *reinterpret_cast<const float4*>(zr + c);
+        keep[i] = make_float4(a.x * silu_f(b.x), a.y * silu_f(b.y), a.z * silu_f(b.z), a.w * silu_f(b.w));
+        ss = fmaf(keep[i].x, keep[i].x, fmaf(keep[i].y, keep[i].y, fmaf(keep[i].z, keep[i].z, fmaf(keep[i].w, keep[i].w, ss))));
+    }
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)gs + eps);
+    TO* yr = y + (size_t)blockIdx.y * ldy + c0;
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        if (c >= gs) continue;
+        const float4 wv = *reinterpret_cast<const float4*>(w + c0 + c);
+        TO v[4] = {from_f32<TO>(keep[i].x * r * wv.x), from_f32<TO>(keep[i].y * r * wv.y), from_f32<TO>(keep[i].z * r * wv.z),
+                   from_f32<TO>(keep[i].w * r * wv.w)};
+        if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(yr + c) = *reinterpret_cast<const float4*>(v);
+        else *reinterpret_cast<uint2*>(yr + c) = *reinterpret_cast<const uint2*>(v);
+    }
+}
+
+template <typename TO>
+static cudaError_t silu_gate_launch(const float* o, long long ldo, const float* z, long long ldz, const float* w, TO* y, long long ldy,
+                                    int T, int groups, int gs, float eps, bool pdl, cudaStream_t st) {
+    auto al = [](const void* q, int b) { return (reinterpret_cast<uintptr_t>(q) & (b - 1)) == 0; };
+    // (few tokens have no warps to spare: a CTA per part)
+    if (T > 64 && gs % 4 == 0 && gs <= 1024 && ldo % 4 == 0 && ldz % 4 == 0 && ldy % 4 == 0 && al(o, 16) && al(z, 16) && al(w, 16) &&
+        al(y, 4 * (int)sizeof(TO))) {
+        const dim3 grid(cdiv(groups, 8), T), block(256);
+        if (gs <= 256) return launch(k_silu_gate_group_rmsnorm_warp<TO, 2>, grid, block, 0, st, pdl, o, ldo, z, ldz, w, y, ldy, groups, gs, eps);
+        if (gs <= 512) return launch(k_silu_gate_group_rmsnorm_warp<TO, 4>, grid, block, 0, st, pdl, o, ldo, z, ldz, w, y, ldy, groups, gs, eps);
+        return launch(k_silu_gate_group_rmsnorm_warp<TO, 8>, grid, block, 0, st, pdl, o, ldo, z, ldz, w, y, ldy, groups, gs, eps);
+    }
+    return launch(k_silu_gate_group_rmsnorm<TO>, dim3(groups, T), dim3(gs >= 2048 ? 512 : (gs >= 512 ? 256 : 128)), 0, st, pdl, o, ldo, z,
+                  ldz, w, y, ldy, gs, eps);
+}
+
 }  // namespace zl
 
 using namespace zl;
@@ -351,20 +572,22 @@ extern "C" int zl_ssm_scan(const float* proj, long long ld, int col_x, int col_d
     ZL_CHECK_ARG(al16(workspace));
     p.vec = C % 4 == 0 && inner % 4 == 0 && vdim % 4 == 0 && state % 4 == 0;
     const bool v4 = C % 4 == 0 && ld % 4 == 0 && col_x % 4 == 0 && al16(proj) && al16(conv_weight);
-    const dim3 grid(cdiv(C, 256 * (v4 ? 4 : 1)) + 1, T);
-    if (v4) ZL_CHECK_CUDA(launch(k_ssm_prep<4>, grid, dim3(256), 0, stream, pdl != 0, p));
-    else ZL_CHECK_CUDA(launch(k_ssm_prep<1>, grid, dim3(256), 0, stream, pdl != 0, p));
-    switch (state <= 128 ? (state + 15) / 16 : (state <= 192 ? 12 : (state <= 256 ? 16 : 0))) {
-        case 1: return ssm_launch<1>(p, runs, pdl != 0, stream);
-        case 2: return ssm_launch<2>(p, runs, pdl != 0, stream);
-        case 3: return ssm_launch<3>(p, runs, pdl != 0, stream);
-        case 4: return ssm_launch<4>(p, runs, pdl != 0, stream);
-        case 5: return ssm_launch<5>(p, runs, pdl != 0, stream);
-        case 6: return ssm_launch<6>(p, runs, pdl != 0, stream);
-        case 7: return ssm_launch<7>(p, runs, pdl != 0, stream);
-        case 8: return ssm_launch<8>(p, runs, pdl != 0, stream);
-        case 12: return ssm_launch<12>(p, runs, pdl != 0, stream);
-        case 16: return ssm_launch<16>(p, runs, pdl != 0, stream);
+    ZL_CHECK_CUDA(v4 ? ssm_prep_launch<4>(p, T, pdl != 0, stream) : ssm_prep_launch<1>(p, T, pdl != 0, stream));
+    if (runs == T && state <= 256) {   // a token per sequence
+        const dim3 grid(cdiv(vdim, 16), heads, runs), block(128);
+        if (state <= 32) ZL_CHECK_CUDA(launch(k_ssm_step<1>, grid, block, 0, stream, pdl != 0, p));
+        else if (state <= 64) ZL_CHECK_CUDA(launch(k_ssm_step<2>, grid, block, 0, stream, pdl != 0, p));
+        else if (state <= 128) ZL_CHECK_CUDA(launch(k_ssm_step<4>, grid, block, 0, stream, pdl != 0, p));
+        else ZL_CHECK_CUDA(launch(k_ssm_step<8>, grid, block, 0, stream, pdl != 0, p));
+        return ZL_OK;
+    }
+    switch (state <= 128 ? (state + 31) / 32 : (state <= 192 ? 6 : (state <= 256 ? 8 : 0))) {
+        case 1: return ssm_launch<1, 8, 2>(p, runs, pdl != 0, stream);
+        case 2: return ssm_launch<2, 8, 2>(p, runs, pdl != 0, stream);
+        case 3: return ssm_launch<3, 8, 2>(p, runs, pdl != 0, stream);
+        case 4: return ssm_launch<4, 8, 2>(p, runs, pdl != 0, stream);
+        case 6: return ssm_launch<6, 8, 2>(p, runs, pdl != 0, stream);
+        case 8: return ssm_launch<8, 8, 2>(p, runs, pdl != 0, stream);
         default: break;
     }
     const size_t smem = (size_t)state * 32 * sizeof(float);
@@ -383,15 +606,11 @@ extern "C" int zl_silu_gate_group_rmsnorm(const float* o, long long ldo, const f
     ZL_CHECK_ARG(o && z && weight && y && T > 0 && T <= 65535 && D > 0 && groups > 0 && D % groups == 0);
     ZL_CHECK_ARG(ldo >= D && ldz >= D && ldy >= D && (out_dtype == ZL_F16 || out_dtype == ZL_BF16 || out_dtype == ZL_F32));
     const int gs = D / groups;
-    const dim3 grid(groups, T), block(gs >= 2048 ? 512 : (gs >= 512 ? 256 : 128));
     cudaError_t e;
-    if (out_dtype == ZL_F32)
-        e = launch(k_silu_gate_group_rmsnorm<float>, grid, block, 0, stream, pdl != 0, o, ldo, z, ldz, weight, (float*)y, ldy, gs, eps);
+    if (out_dtype == ZL_F32) e = silu_gate_launch(o, ldo, z, ldz, weight, (float*)y, ldy, T, groups, gs, eps, pdl != 0, stream);
     else if (out_dtype == ZL_BF16)
-        e = launch(k_silu_gate_group_rmsnorm<__nv_bfloat16>, grid, block, 0, stream, pdl != 0, o, ldo, z, ldz, weight, (__nv_bfloat16*)y,
-                   ldy, gs, eps);
-    else
-        e = launch(k_silu_gate_group_rmsnorm<__half>, grid, block, 0, stream, pdl != 0, o, ldo, z, ldz, weight, (__half*)y, ldy, gs, eps);
+        e = silu_gate_launch(o, ldo, z, ldz, weight, (__nv_bfloat16*)y, ldy, T, groups, gs, eps, pdl != 0, stream);
+    else e = silu_gate_launch(o, ldo, z, ldz, weight, (__half*)y, ldy, T, groups, gs, eps, pdl != 0, stream);
     ZL_CHECK_CUDA(e);
     return ZL_OK;
 }
