@@ -355,7 +355,7 @@ def test_latent_rows_with_scaled_rotation(cuda, lib, dtype):
     assert (row[:, R:RC] == 5).all() and (row[:, RC + r:] == 5).all() and bool((cache[1, 36] == 5).all())
 
 
-@pytest.mark.parametrize("shape", [(6, 32, 48, 2, 3), (4, 5, 9, 2, 4), (2, 64, 128, 1, 4), (3, 40, 20, 3, 2), (1, 1, 1, 1, 1), (8, 16, 256, 4, 4),
+@pytest.mark.parametrize("shape", [(6, 48, 40, 3, 3), (4, 5, 9, 2, 4), (2, 64, 128, 1, 4), (3, 40, 20, 3, 2), (1, 1, 1, 1, 1), (8, 16, 256, 4, 4),
                                    (2, 34, 96, 2, 7), (2, 12, 272, 1, 3), (4, 8, 64, 4, 1)])
 def test_state_space_scan(cuda, lib, shape):
     """Convolution, step sizes, decays and the recurrence over a plan of portions and single tokens of three sequences on slots full
